@@ -53,6 +53,11 @@ struct AttnArgs {
     int keep_first;                    // under a window: the first keys of a sequence (positions below this) stay
                                        // visible to every later query, each where it was written; 0: none
     float scale_log2e;
+    float cap_log2e, scale_over_cap;   // a soft cap on the scores: cap * tanh(scale q.k / cap) in base-2 units is
+                                       // cap_log2e * tanh(scale_over_cap * q.k); cap_log2e 0: none
+    const float* head_gate;            // [rows, query heads] or nullptr: every head's output is multiplied by sigmoid of
+    long gate_stride;                  // its number, which arrives as gate_partials float32 shares (added first)
+    int gate_partials; long gate_partial_stride;
     const float* score_slopes;         // per query head, or nullptr: slope * (key position - query position) is added
                                        // to the scaled score (a linear penalty on distance; <= 0 for the keys a
                                        // query sees when the slope is >= 0)
@@ -76,6 +81,13 @@ struct AttnArgs {
 // What a head's sink adds to a row's denominator whose terms are 2^(score - m), scores in base-2 units.
 __device__ __forceinline__ float sink_term(const AttnArgs& a, int head, float m) {
     return (a.sinks && m > -INFINITY) ? exp2f(a.sinks[head] * 1.4426950408889634f - m) : 0.0f;
+}
+
+// What a head's gate multiplies the output of (row, head) with.
+__device__ __forceinline__ float head_gate_factor(const AttnArgs& a, int row, int head) {
+    if (!a.head_gate) return 1.0f;
+    return 1.0f / (1.0f + expf(-fb_slab_sum(a.head_gate + (size_t)row * a.gate_stride, head, a.gate_partials,
+                                            a.gate_partial_stride)));
 }
 
 // The page id of logical page `logical` of a sequence whose table row `table` starts at logical page `base_page`

@@ -278,6 +278,15 @@ attention_mma_kernel(const __grid_constant__ AttnArgs a) {
             }
         }
         // ---- scale, mask, online softmax ----
+        const float to_log2 = a.cap_log2e > 0.0f ? 1.0f : a.scale_log2e;
+        if (a.cap_log2e > 0.0f) {
+#pragma unroll
+            for (int rb = 0; rb < R; ++rb)
+#pragma unroll
+                for (int nb = 0; nb < NSB; ++nb)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) s[rb][nb][e] = fb_softcap(s[rb][nb][e] * a.scale_over_cap, a.cap_log2e);
+        }
         uint32_t pa[R][KT / 16][4];            // the probabilities as A fragments of P V
 #pragma unroll
         for (int rb = 0; rb < R; ++rb) {
@@ -289,7 +298,7 @@ attention_mma_kernel(const __grid_constant__ AttnArgs a) {
                     const int h = e >> 1;
                     const int t = tile_start + nb * 8 + 2 * (lane & 3) + (e & 1);
                     const bool ok = key_seen(t, p_row[rb][h], t0_row[rb][h], kr.keep);
-                    const float v = ok ? fmaf(slope_row[rb][h], (float)(t - p_row[rb][h]), s[rb][nb][e] * a.scale_log2e) : -INFINITY;
+                    const float v = ok ? fmaf(slope_row[rb][h], (float)(t - p_row[rb][h]), s[rb][nb][e] * to_log2) : -INFINITY;
                     s[rb][nb][e] = v;
                     tile_max[h] = fmaxf(tile_max[h], v);
                 }
@@ -375,7 +384,7 @@ attention_mma_kernel(const __grid_constant__ AttnArgs a) {
             if (r >= rows_valid) continue;
             const int token = q_start + tok0 + r / G, head = kvh * G + r % G;
             const float l_all = l_run[rb][h] + sink_term(a, head, m_run[rb][h]);
-            const float inv = l_all > 0.0f ? 1.0f / l_all : 0.0f;
+            const float inv = (l_all > 0.0f ? 1.0f / l_all : 0.0f) * head_gate_factor(a, token, head);
             __nv_bfloat16* dst = a.out + (size_t)token * a.out_stride + (size_t)head * hd;
 #pragma unroll
             for (int d = 0; d < NDB; ++d) {
@@ -452,6 +461,8 @@ FB_API void fb_set_attention_tc(int on) { g_attention_tc = on ? 1 : 0; }
 // sequence's table row stands for; multi_seqs (may be null: all sequences): the n_multi sequences that bring more
 // than one token, which is all that the arrangements for portions lay their grid over.  max_q_len / max_kv_len / any_short / any_long come from the host's copy of the
 // step descriptor.  `scratch` holds the arrival counters and partial results of the split-key arrangement.
+// softcap > 0: scores are softcap * tanh(scale q.k / softcap).  head_gate (may be null): float32 [rows, nh], rows
+// gate_stride apart, the first of gate_partials shares; every head's output is multiplied by sigmoid of its number.
 // prefetch_*: the first prefetch_bytes_per_row bytes of each of prefetch_rows rows (prefetch_row_stride bytes
 // apart, from prefetch_base) are fetched into L2 when the split-key kernel's stream of cache ends: the matrix of
 // the product that follows (a hint; null base: none).
@@ -460,8 +471,9 @@ FB_API int fb_paged_attention_mma(const void* q, long long q_stride, void* out, 
                                   const int* block_table, int table_stride, const int* table_base, int table_head,
                                   const int* seq_q_start, const int* seq_q_len, const int* seq_pos_start,
                                   const int* multi_seqs, int n_multi, int n_seqs, int max_q_len, int max_kv_len, int any_short, int any_long, int nh, int nkv, int hd,
-                                  int window, int keep_first, float scale, const float* score_slopes, const float* sinks,
-                                  int weights_hi_lo, float* scratch,
+                                  int window, int keep_first, float scale, float softcap, const float* score_slopes,
+                                  const float* sinks, const float* head_gate, long long gate_stride, int gate_partials,
+                                  long long gate_partial_stride, int weights_hi_lo, float* scratch,
                                   long long scratch_floats,
                                   const void* prefetch_base, long long prefetch_rows, long long prefetch_row_stride,
                                   int prefetch_bytes_per_row, int* status, cudaStream_t stream) {
@@ -474,6 +486,7 @@ FB_API int fb_paged_attention_mma(const void* q, long long q_stride, void* out, 
     FB_REQUIRE(q_stride % 8 == 0 && ((uintptr_t)q & 15) == 0, "attention_mma: q rows must be 16-byte aligned");
     FB_REQUIRE(out_stride % 2 == 0 && ((uintptr_t)out & 3) == 0, "attention_mma: out rows must be 4-byte aligned");
     FB_REQUIRE(page_size > 0 && n_pages > 0 && window >= 0 && keep_first >= 0, "attention_mma: bad cache geometry");
+    FB_REQUIRE(softcap >= 0.0f && (!head_gate || gate_stride >= nh), "attention_mma: bad cap or gate");
     if (n_seqs == 0) return 0;
     const int HD_MAX = hd <= 32 ? 32 : hd <= 64 ? 64 : hd <= 128 ? 128 : 256;
     AttnArgs a;
@@ -488,6 +501,10 @@ FB_API int fb_paged_attention_mma(const void* q, long long q_stride, void* out, 
     a.nh = nh; a.nkv = nkv; a.hd = hd; a.window = window;
     a.keep_first = window > 0 ? keep_first : 0;
     a.scale_log2e = scale * 1.4426950408889634f;
+    a.cap_log2e = softcap > 0.0f ? softcap * 1.4426950408889634f : 0.0f;
+    a.scale_over_cap = softcap > 0.0f ? scale / softcap : 0.0f;
+    a.head_gate = head_gate; a.gate_stride = (long)gate_stride;
+    a.gate_partials = gate_partials < 1 ? 1 : gate_partials; a.gate_partial_stride = (long)gate_partial_stride;
     a.score_slopes = score_slopes;
     a.sinks = sinks;
     a.weights_hi_lo = weights_hi_lo ? 1 : 0;

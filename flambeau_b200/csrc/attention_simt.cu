@@ -16,6 +16,9 @@
 // Value rows may be narrower or wider than key rows (vd against hd).  With `sinks` (one float32 per query head) the
 // softmax has one more slot whose score is that number as it stands (not scaled) and which carries no value: it
 // enters the running maximum and the denominator once, and nothing else.
+//
+// softcap > 0: scores are softcap * tanh(scale q.k / softcap).  head_gate (float32 [rows, nh], possibly shares): every
+// head's output is multiplied by sigmoid of its number.
 #include "common.cuh"
 
 template <typename T, int NDR>   // NDR = ceil(value size / 32) accumulator registers per lane
@@ -25,8 +28,10 @@ paged_attention_simt_kernel(const T* __restrict__ q, long q_stride, T* __restric
                             int n_pages, const int* __restrict__ block_table, int table_stride,
                             const int* __restrict__ table_base, int table_head,
                             const int* __restrict__ positions, const int* __restrict__ row_seq, int n, int nh,
-                            int nkv, int hd, int vd, int window, int keep_first, float scale,
-                            const float* __restrict__ score_slopes, const float* __restrict__ sinks, int* status) {
+                            int nkv, int hd, int vd, int window, int keep_first, float scale, float softcap,
+                            const float* __restrict__ score_slopes, const float* __restrict__ sinks,
+                            const float* __restrict__ head_gate, long gate_stride, int gate_partials,
+                            long gate_partial_stride, int* status) {
     fb_pdl_launch_dependents();
     fb_pdl_wait();
     extern __shared__ float q_sh[];                    // [4 warps][hd]
@@ -74,7 +79,9 @@ paged_attention_simt_kernel(const T* __restrict__ q, long q_stride, T* __restric
                 const T* kr = k_pool + (((size_t)my_page * nkv + kvh) * page_size + (t % page_size)) * hd;
                 float dot = 0.0f;
                 for (int d = 0; d < hd; ++d) dot = fmaf(qs[d], fb_to_float(kr[d]), dot);
-                s = dot * scale + slope * (float)(t - p);
+                s = dot * scale;
+                if (softcap > 0.0f) s = softcap * tanhf(s / softcap);
+                s += slope * (float)(t - p);
             }
         }
         const float tile_max = fb_warp_max(s);
@@ -109,7 +116,9 @@ paged_attention_simt_kernel(const T* __restrict__ q, long q_stride, T* __restric
 #pragma unroll
         for (int r = 0; r < NDR; ++r) acc[r] *= corr;
     }
-    const float inv = l > 0.0f ? 1.0f / l : 0.0f;
+    float inv = l > 0.0f ? 1.0f / l : 0.0f;
+    if (head_gate)                                      // the head's output times sigmoid of its gate
+        inv /= 1.0f + expf(-fb_slab_sum(head_gate + (size_t)row * gate_stride, head, gate_partials, gate_partial_stride));
     T* op = out + (size_t)row * out_stride + (size_t)head * vd;
 #pragma unroll
     for (int r = 0; r < NDR; ++r) {
@@ -123,14 +132,15 @@ static int launch_attention_simt(const void* q, long q_stride, void* out, long o
                                  const void* v_pool, int page_size, int n_pages, const int* block_table,
                                  int table_stride, const int* table_base, int table_head, const int* positions, const int* row_seq,
                                  int n, int nh,
-                                 int nkv, int hd, int vd, int window, int keep_first, float scale, const float* score_slopes,
-                                 const float* sinks, int* status, cudaStream_t stream) {
+                                 int nkv, int hd, int vd, int window, int keep_first, float scale, float softcap,
+                                 const float* score_slopes, const float* sinks, const float* head_gate, long gate_stride,
+                                 int gate_partials, long gate_partial_stride, int* status, cudaStream_t stream) {
     const long items = (long)n * nh;
     const unsigned blocks = (unsigned)((items + 3) / 4);
     fb_launch((paged_attention_simt_kernel<T, NDR>), blocks, 128, 4 * hd * sizeof(float), stream, 
         (const T*)q, q_stride, (T*)out, out_stride, (const T*)k_pool, (const T*)v_pool, page_size, n_pages,
-        block_table, table_stride, table_base, table_head, positions, row_seq, n, nh, nkv, hd, vd, window, keep_first, scale, score_slopes, sinks,
-        status);
+        block_table, table_stride, table_base, table_head, positions, row_seq, n, nh, nkv, hd, vd, window, keep_first, scale,
+        softcap, score_slopes, sinks, head_gate, gate_stride, gate_partials, gate_partial_stride, status);
     return fb_check_launch("paged_attention_simt");
 }
 
@@ -138,18 +148,23 @@ FB_API int fb_paged_attention_simt(const void* q, long long q_stride, void* out,
                                    const void* k_pool, const void* v_pool, int page_size, int n_pages,
                                    const int* block_table, int table_stride, const int* table_base, int table_head,
                                    const int* positions, const int* row_seq, int n, int nh, int nkv, int hd,
-                                   int vd, int window, int keep_first, float scale, const float* score_slopes, const float* sinks,
-                                   int* status, cudaStream_t stream) {
+                                   int vd, int window, int keep_first, float scale, float softcap,
+                                   const float* score_slopes, const float* sinks, const float* head_gate,
+                                   long long gate_stride, int gate_partials, long long gate_partial_stride, int* status,
+                                   cudaStream_t stream) {
     if (vd <= 0) vd = hd;
     FB_REQUIRE(n >= 0 && nh > 0 && nkv > 0 && hd > 0, "attention: bad sizes n=%d heads=%d kv=%d hd=%d", n, nh, nkv, hd);
     FB_REQUIRE(nh % nkv == 0, "attention: %d query heads are not a multiple of %d key/value heads", nh, nkv);
     FB_REQUIRE(hd <= 512 && vd <= 512, "attention: head size %d / value size %d is larger than 512", hd, vd);
     FB_REQUIRE(page_size > 0 && n_pages > 0 && window >= 0 && keep_first >= 0, "attention: bad cache geometry");
+    FB_REQUIRE(softcap >= 0.0f && (!head_gate || gate_stride >= nh), "attention: bad cap or gate");
     if (n == 0) return 0;
+    if (gate_partials < 1) gate_partials = 1;
 #define FB_ATTN_CASE(NDR)                                                                                      \
     FB_DISPATCH_DTYPE(dtype, T, return (launch_attention_simt<T, NDR>(q, (long)q_stride, out, (long)out_stride,     \
         k_pool, v_pool, page_size, n_pages, block_table, table_stride, table_base, table_head, positions, row_seq, n, nh, \
-        nkv, hd, vd, window, keep_first, scale, score_slopes, sinks, status, stream)))
+        nkv, hd, vd, window, keep_first, scale, softcap, score_slopes, sinks, head_gate, (long)gate_stride, gate_partials, \
+        (long)gate_partial_stride, status, stream)))
     if (vd <= 32) { FB_ATTN_CASE(1); }
     else if (vd <= 64) { FB_ATTN_CASE(2); }
     else if (vd <= 128) { FB_ATTN_CASE(4); }

@@ -84,7 +84,7 @@ __device__ __forceinline__ void short_prefix(const AttnArgs& a, int G, const Sho
 // of the head's columns.  The partials were written by other SMs: they are read past the L1.
 template <int HD_MAX>
 __device__ __forceinline__ void merge_row(const AttnArgs& a, size_t slot0, int n_chunks, int r, int lane,
-                                          __nv_bfloat16* dst, int head) {
+                                          __nv_bfloat16* dst, int row, int head) {
     constexpr int U = HD_MAX <= 128 ? 16 : 8;          // partials whose loads are in flight together
     float acc[HD_MAX / 32];
 #pragma unroll
@@ -124,7 +124,7 @@ __device__ __forceinline__ void merge_row(const AttnArgs& a, size_t slot0, int n
         }
     }
     l = fb_warp_sum(l) + sink_term(a, head, m);
-    const float inv = l > 0.0f ? 1.0f / l : 0.0f;
+    const float inv = (l > 0.0f ? 1.0f / l : 0.0f) * head_gate_factor(a, row, head);
 #pragma unroll
     for (int i = 0; i < HD_MAX / 32; ++i) {
         const int d = lane + 32 * i;
@@ -439,6 +439,13 @@ attention_split_kernel(const __grid_constant__ AttnArgs a) {
                     }
                 }
                 // ---- scale, mask, online softmax ----
+                const float to_log2 = a.cap_log2e > 0.0f ? 1.0f : a.scale_log2e;
+                if (a.cap_log2e > 0.0f) {
+#pragma unroll
+                    for (int nb = 0; nb < 2; ++nb)
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) s[nb][e] = fb_softcap(s[nb][e] * a.scale_over_cap, a.cap_log2e);
+                }
                 float tile_max[2] = {-INFINITY, -INFINITY};
 #pragma unroll
                 for (int nb = 0; nb < 2; ++nb)
@@ -447,7 +454,7 @@ attention_split_kernel(const __grid_constant__ AttnArgs a) {
                         const int h = e >> 1;
                         const int t = tile_start + key0 + nb * 8 + 2 * (lane & 3) + (e & 1);
                         const bool ok = key_seen(t, p_row[h], t0_row[h], cur.kr.keep);
-                        const float v = ok ? fmaf(slope_row[h], (float)(t - p_row[h]), s[nb][e] * a.scale_log2e) : -INFINITY;
+                        const float v = ok ? fmaf(slope_row[h], (float)(t - p_row[h]), s[nb][e] * to_log2) : -INFINITY;
                         s[nb][e] = v;
                         tile_max[h] = fmaxf(tile_max[h], v);
                     }
@@ -569,7 +576,7 @@ attention_split_kernel(const __grid_constant__ AttnArgs a) {
                     } else {                          // the whole pair was this CTA's: the result itself
                         const int token = q_start + r / G, head = kvh * G + r % G;
                         const float l_sink = l_all[h] + sink_term(a, head, m_all[h]);
-                        const float inv = l_sink > 0.0f ? 1.0f / l_sink : 0.0f;
+                        const float inv = (l_sink > 0.0f ? 1.0f / l_sink : 0.0f) * head_gate_factor(a, token, head);
                         __nv_bfloat16* dst = a.out + (size_t)token * a.out_stride + (size_t)head * hd + 2 * (lane & 3);
 #pragma unroll
                         for (int d = 0; d < NDB; ++d) {
@@ -597,7 +604,7 @@ attention_split_kernel(const __grid_constant__ AttnArgs a) {
                 for (int r = warp; r < rows_valid; r += SPLIT_SCORERS) {
                     const int token = q_start + r / G, head = kvh * G + r % G;
                     merge_row<HD_MAX>(a, slot0, cur.n_chunks, r, lane,
-                                      a.out + (size_t)token * a.out_stride + (size_t)head * hd, head);
+                                      a.out + (size_t)token * a.out_stride + (size_t)head * hd, token, head);
                 }
             }
         }

@@ -49,14 +49,29 @@ constexpr double FB_MODEL_SM_FLOPS = 9.0e12;
 
 // ---- activations of gated feed-forwards -----------------------------------------
 // out = act(gate) * up.  The code travels as a launcher argument (0 = no gating where that is an option).
-enum FbAct : int { FB_ACT_SILU = 1, FB_ACT_GELU_TANH = 2 };
-inline bool fb_act_known(int act) { return act == FB_ACT_SILU || act == FB_ACT_GELU_TANH; }
-__device__ __forceinline__ float fb_gate_times(int act, float g, float u) {
-    if (act == FB_ACT_GELU_TANH) {
-        // 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3)))
-        const float t = tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g));
-        return 0.5f * g * (1.0f + t) * u;
+// FB_ACT_LIMITED cuts both operands off and shifts the up side: with g = min(gate, limit) and u = up held to
+// [-limit, limit], out = g sigmoid(slope g) (u + 1); `limit` and `slope` travel beside the code and mean nothing to the
+// other activations.
+enum FbAct : int { FB_ACT_SILU = 1, FB_ACT_GELU_TANH = 2, FB_ACT_LIMITED = 3 };
+struct FbGate {
+    int act;               // an FbAct code, 0: no gating
+    float limit, slope;
+};
+inline bool fb_act_known(int act) { return act >= FB_ACT_SILU && act <= FB_ACT_LIMITED; }
+inline bool fb_gate_known(const FbGate& gate) {
+    return fb_act_known(gate.act) && (gate.act != FB_ACT_LIMITED || gate.limit > 0.0f);
+}
+__device__ __forceinline__ float fb_gelu_tanh(float z) {
+    // 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))
+    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+__device__ __forceinline__ float fb_gate_times(const FbGate& gate, float g, float u) {
+    if (gate.act == FB_ACT_LIMITED) {
+        g = fminf(g, gate.limit);
+        u = fminf(fmaxf(u, -gate.limit), gate.limit);
+        return g / (1.0f + expf(-gate.slope * g)) * (u + 1.0f);
     }
+    if (gate.act == FB_ACT_GELU_TANH) return fb_gelu_tanh(g) * u;
     return g / (1.0f + expf(-g)) * u;             // SiLU (crates/model-ops/src/ops/activation.rs:107-118)
 }
 
@@ -67,7 +82,7 @@ inline bool fb_plain_act_known(int act) { return act >= FB_PLAIN_NONE && act <= 
 __device__ __forceinline__ float fb_plain_act(int act, float z) {
     if (act == FB_PLAIN_RELU_SQUARED) { const float r = fmaxf(z, 0.0f); return r * r; }
     if (act == FB_PLAIN_SILU) return z / (1.0f + expf(-z));
-    if (act == FB_PLAIN_GELU_TANH) return fb_gate_times(FB_ACT_GELU_TANH, z, 1.0f);
+    if (act == FB_PLAIN_GELU_TANH) return fb_gelu_tanh(z);
     return z;
 }
 
@@ -148,6 +163,19 @@ template <typename T> __device__ __forceinline__ T fb_from_float(float v);
 template <> __device__ __forceinline__ float fb_from_float<float>(float v) { return v; }
 template <> __device__ __forceinline__ __nv_bfloat16 fb_from_float<__nv_bfloat16>(float v) {
     return __float2bfloat16_rn(v);
+}
+
+// ---- scores that pass a soft cap ---------------------------------------------------
+// cap * tanh(y) with y = score / cap, for kernels whose scores are in units of their own (`cap` in the same).  For large
+// |y| from one exponential, (1 - e) / (1 + e) with e = 2^(-2 log2(e) |y|); for small |y|, where 1 - e cancels, the Taylor
+// series to y^7, whose next term is below 6e-8 of the result at the border.
+__device__ __forceinline__ float fb_softcap(float y, float cap) {
+    const float a = fabsf(y);
+    const float e = exp2f(-2.8853900817779268f * a);
+    const float big = __fdividef(1.0f - e, 1.0f + e);
+    const float q = y * y;
+    const float small = a * fmaf(q, fmaf(q, fmaf(q, -17.0f / 315.0f, 2.0f / 15.0f), -1.0f / 3.0f), 1.0f);
+    return copysignf(cap * (a < 0.2f ? small : big), y);
 }
 
 // ---- reductions -------------------------------------------------------------

@@ -2,7 +2,7 @@
 // residual add + RMSNorm, rotary tables, rotary + paged cache write, act(gate)*up.
 // All arithmetic is float32 whatever the storage type; the residual stream
 // itself is float32 in both engine modes.
-#include "common.cuh"
+#include "rows.cuh"
 
 // ---------------------------------------------------------------------------
 // Embedding: x[t,:] = E[ids[t],:] * scale  (crates/forward/src/core/composites/embed.rs:26-62; scale 1 there)
@@ -74,27 +74,6 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ x, const TD* __restrict__
 
 // Fast path: width a multiple of 4 and at most 4 * VPT * blockDim: every thread keeps its part of the row in
 // registers and issues all of its loads before the first use, so a row costs one round trip to memory.
-template <typename T> struct Vec4 {};
-template <> struct Vec4<float> {
-    static __device__ __forceinline__ float4 load(const float* p) { return *reinterpret_cast<const float4*>(p); }
-    static __device__ __forceinline__ void store(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-};
-template <> struct Vec4<__nv_bfloat16> {
-    static __device__ __forceinline__ float4 load(const __nv_bfloat16* p) {
-        const uint2 raw = *reinterpret_cast<const uint2*>(p);
-        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-        const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-        return make_float4(a.x, a.y, b.x, b.y);
-    }
-    static __device__ __forceinline__ void store(__nv_bfloat16* p, float4 v) {
-        __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
-        uint2 raw;
-        raw.x = *reinterpret_cast<uint32_t*>(&a);
-        raw.y = *reinterpret_cast<uint32_t*>(&b);
-        *reinterpret_cast<uint2*>(p) = raw;
-    }
-};
-
 template <typename TD, typename TW, typename TO, int VPT>
 __global__ void __launch_bounds__(1024)
 add_rmsnorm_vec_kernel(float* __restrict__ x, const TD* __restrict__ delta, int n_partials,
@@ -528,21 +507,6 @@ FB_API int fb_rope_table(const int* positions, const double* inv_freq, float* co
 // crates/kernels-hip/src/kernels/rope_neox_partial_f16.cu:39-52 (rotation),
 // kv_append_f16_paged_prefill.cu (row placement).
 // ---------------------------------------------------------------------------
-// Element j of a row that is stored as `n_partials` slabs `partial_stride` elements apart (split-K shares).
-template <typename TI>
-__device__ __forceinline__ float slab_sum(const TI* __restrict__ row, int j, int n_partials, long partial_stride) {
-    float acc = fb_to_float(row[j]);
-    for (int p = 1; p < n_partials; p += 8) {         // eight independent loads in flight, added in slab order
-        float a[8];
-#pragma unroll
-        for (int u = 0; u < 8; ++u)
-            a[u] = p + u < n_partials ? fb_to_float(row[(size_t)(p + u) * partial_stride + j]) : 0.0f;
-#pragma unroll
-        for (int u = 0; u < 8; ++u) acc += a[u];
-    }
-    return acc;
-}
-
 template <typename TI, typename T>
 __global__ void rope_kv_write_kernel(const TI* __restrict__ q_in, long q_in_stride, int n_partials,
                                      long partial_stride, T* __restrict__ q_out,
@@ -610,20 +574,6 @@ __global__ void rope_kv_write_kernel(const TI* __restrict__ q_in, long q_in_stri
 // The same work four elements at a time (all strides, the head size and the rotary half multiples of 4,
 // 16-byte aligned rows): one item = four consecutive pairs of one head, or four untouched dimensions, or four
 // values.  Items of a token: (nh + nkv) * (hd - half) / 4 rotary items, then nkv * hd / 4 value items.
-template <typename TI>
-__device__ __forceinline__ float4 slab_sum4(const TI* __restrict__ p, int n_partials, long partial_stride) {
-    float4 acc = Vec4<TI>::load(p);
-    for (int s = 1; s < n_partials; s += 8) {         // eight independent loads in flight, added in slab order
-        float4 a[8];
-#pragma unroll
-        for (int u = 0; u < 8; ++u)
-            a[u] = s + u < n_partials ? Vec4<TI>::load(p + (size_t)(s + u) * partial_stride) : make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-        for (int u = 0; u < 8; ++u) { acc.x += a[u].x; acc.y += a[u].y; acc.z += a[u].z; acc.w += a[u].w; }
-    }
-    return acc;
-}
-
 // TOK tokens per thread (the same item of each): every load of the thread's tokens is issued before the first
 // use, which is what fills the memory pipe when a prompt's portion brings thousands of tokens.  A token past the
 // end reads the last token again and stores nothing.
@@ -785,7 +735,7 @@ FB_API int fb_rope_kv_write(const void* q_in, long long q_in_stride, int n_parti
 // ---------------------------------------------------------------------------
 template <typename TI, typename T>
 __global__ void gate_mul_kernel(const TI* __restrict__ gu, long stride, int n_partials, long partial_stride,
-                                T* __restrict__ out, int n, int I, int act) {
+                                T* __restrict__ out, int n, int I, FbGate act) {
     fb_pdl_launch_dependents();
     fb_pdl_wait();
     const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -800,7 +750,7 @@ __global__ void gate_mul_kernel(const TI* __restrict__ gu, long stride, int n_pa
 // Two outputs per thread from one 4-wide load (g0, u0, g1, u1); I even, strides multiples of 4, aligned rows.
 template <typename TI, typename T>
 __global__ void gate_mul_vec_kernel(const TI* __restrict__ gu, long stride, int n_partials, long partial_stride,
-                                    T* __restrict__ out, int n, int I, int act) {
+                                    T* __restrict__ out, int n, int I, FbGate act) {
     fb_pdl_launch_dependents();
     fb_pdl_wait();
     const int nvec = I >> 1;
@@ -814,12 +764,13 @@ __global__ void gate_mul_vec_kernel(const TI* __restrict__ gu, long stride, int 
 }
 
 // gate_up has dtype in_dtype and may be split-K shares (n_partials slabs partial_stride elements apart);
-// out has dtype out_dtype; `act` is an FbAct code.
+// out has dtype out_dtype; `act_code` is an FbAct code with its constants behind it.
 FB_API int fb_gate_mul(const void* gate_up, long long stride, int in_dtype, int n_partials,
-                       long long partial_stride, void* out, int out_dtype, int n, int I, int act,
-                       cudaStream_t stream) {
+                       long long partial_stride, void* out, int out_dtype, int n, int I, int act_code, float limit,
+                       float slope, cudaStream_t stream) {
+    const FbGate act = {act_code, limit, slope};
     FB_REQUIRE(n >= 0 && I > 0 && stride >= 2LL * I, "gate_mul: bad sizes n=%d I=%d stride=%lld", n, I, stride);
-    FB_REQUIRE(fb_act_known(act), "gate_mul: unknown activation code %d", act);
+    FB_REQUIRE(fb_gate_known(act), "gate_mul: unknown activation code %d, or its limit is not positive", act_code);
     if (n == 0) return 0;
     if (n_partials < 1) n_partials = 1;
     const bool vec = I % 2 == 0 && stride % 4 == 0 && partial_stride % 4 == 0 && (uintptr_t)gate_up % 16 == 0;
@@ -934,23 +885,40 @@ FB_API int fb_sigmoid_gate(void* a, long long a_stride, int dtype, const float* 
 }
 
 // ---------------------------------------------------------------------------
-// x[r, :] += v[:] for the first n rows of the float32 stream (a learned vector that joins every token alike).
+// x[r, :] += v[:] for the first n rows of the float32 stream (a learned vector that joins every token alike), and
+// x[r, :] += y[r, :] of a second stream where there is one (added first).  Either may be absent.
 // ---------------------------------------------------------------------------
-template <typename TW>
-__global__ void add_row_kernel(float* __restrict__ x, const TW* __restrict__ v, int n, int H) {
+template <typename TW, int VEC>
+__global__ void __launch_bounds__(256)
+add_row_kernel(float* __restrict__ x, const float* __restrict__ y, const TW* __restrict__ v, size_t items, int H) {
     fb_pdl_launch_dependents();
     fb_pdl_wait();
-    const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (idx >= (size_t)n * H) return;
-    x[idx] += fb_to_float(v[idx % H]);
+    const size_t idx = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+    if (idx >= items) return;
+    const int c = (int)(idx % H);
+    if constexpr (VEC == 4) {
+        float4 a = Vec4<float>::load(x + idx);
+        if (y) { const float4 b = Vec4<float>::load(y + idx); a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w; }
+        if (v) { const float4 b = Vec4<TW>::load(v + c); a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w; }
+        Vec4<float>::store(x + idx, a);
+    } else {
+        float a = x[idx];
+        if (y) a += y[idx];
+        if (v) a += fb_to_float(v[c]);
+        x[idx] = a;
+    }
 }
 
-FB_API int fb_add_row(float* x, const void* v, int v_dtype, int n, int H, cudaStream_t stream) {
+FB_API int fb_add_row(float* x, const float* y, const void* v, int v_dtype, int n, int H, cudaStream_t stream) {
     FB_REQUIRE(n >= 0 && H > 0, "add_row: bad sizes");
-    if (n == 0) return 0;
+    if (n == 0 || (!y && !v)) return 0;
     const size_t total = (size_t)n * H;
-    FB_DISPATCH_DTYPE(v_dtype, TW,
-        (fb_launch((add_row_kernel<TW>), (unsigned)((total + 255) / 256), 256, 0, stream, x, (const TW*)v, n, H)));
+    const bool vec = H % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)y % 16 == 0 && (uintptr_t)v % 16 == 0;
+    const unsigned blocks = (unsigned)((total / (vec ? 4 : 1) + 255) / 256);
+    FB_DISPATCH_DTYPE(v_dtype, TW, {
+        if (vec) fb_launch((add_row_kernel<TW, 4>), blocks, 256, 0, stream, x, y, (const TW*)v, total, H);
+        else fb_launch((add_row_kernel<TW, 1>), blocks, 256, 0, stream, x, y, (const TW*)v, total, H);
+    });
     return fb_check_launch("add_row");
 }
 
@@ -1021,25 +989,51 @@ FB_API int fb_branch_norm_mix(int count, const float* const* y, const int* n_par
 
 // ---------------------------------------------------------------------------
 // x[r, c] += sum of the shares of delta[r, c]: a part's pending output joins the float32 stream without a norm
-// behind it (for a part that wants the whole stream rather than a normalised copy of it).
+// behind it (for a part that wants the whole stream rather than a normalised copy of it).  `copy` (optional): the rows
+// of the stream as they then are, in the type of a product's operand; without `delta` there is nothing to add and the
+// copy is all that happens.
 // ---------------------------------------------------------------------------
-__global__ void add_slabs_kernel(float* __restrict__ x, const float* __restrict__ delta, int n_partials,
-                                 long partial_stride, size_t total) {
+template <typename TO, int VEC>
+__global__ void __launch_bounds__(256)
+add_slabs_kernel(float* __restrict__ x, const float* __restrict__ delta, int n_partials, long partial_stride,
+                 TO* __restrict__ copy, size_t total) {
     fb_pdl_launch_dependents();
     fb_pdl_wait();
-    const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    const size_t idx = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * VEC;
     if (idx >= total) return;
-    float v = delta[idx];
-    for (int p = 1; p < n_partials; ++p) v += delta[(size_t)p * partial_stride + idx];
-    x[idx] += v;
+    if constexpr (VEC == 4) {
+        float4 v = Vec4<float>::load(x + idx);
+        if (delta) {
+            const float4 d = slab_sum4(delta + idx, n_partials, partial_stride);
+            v.x += d.x; v.y += d.y; v.z += d.z; v.w += d.w;
+            Vec4<float>::store(x + idx, v);
+        }
+        if (copy) Vec4<TO>::store(copy + idx, v);
+    } else {
+        float v = x[idx];
+        if (delta) {
+            v += slab_sum(delta + idx, 0, n_partials, partial_stride);
+            x[idx] = v;
+        }
+        if (copy) copy[idx] = fb_from_float<TO>(v);
+    }
 }
 
-FB_API int fb_add_slabs(float* x, const float* delta, int n_partials, long long partial_stride, int n, int H,
-                        cudaStream_t stream) {
+FB_API int fb_add_slabs(float* x, const float* delta, int n_partials, long long partial_stride, void* copy,
+                        int copy_dtype, int n, int H, cudaStream_t stream) {
     FB_REQUIRE(n >= 0 && H > 0, "add_slabs: bad sizes");
-    if (n == 0) return 0;
+    if (n == 0 || (!delta && !copy)) return 0;
+    if (n_partials < 1) n_partials = 1;
+    if (!copy) copy_dtype = FB_F32;
     const size_t total = (size_t)n * H;
-    fb_launch(add_slabs_kernel, (unsigned)((total + 255) / 256), 256, 0, stream, x, delta,
-              n_partials < 1 ? 1 : n_partials, (long)partial_stride, total);
+    const bool vec = total % 4 == 0 && partial_stride % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)delta % 16 == 0 &&
+                     (uintptr_t)copy % 16 == 0;
+    const unsigned blocks = (unsigned)((total / (vec ? 4 : 1) + 255) / 256);
+    FB_DISPATCH_DTYPE(copy_dtype, TO, {
+        if (vec) fb_launch((add_slabs_kernel<TO, 4>), blocks, 256, 0, stream, x, delta, n_partials, (long)partial_stride,
+                           (TO*)copy, total);
+        else fb_launch((add_slabs_kernel<TO, 1>), blocks, 256, 0, stream, x, delta, n_partials, (long)partial_stride,
+                       (TO*)copy, total);
+    });
     return fb_check_launch("add_slabs");
 }

@@ -76,7 +76,7 @@ __global__ void __launch_bounds__(GEMM_THREADS, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                TO* __restrict__ out, long ldo, long slab_stride, float* __restrict__ partials,
                int* __restrict__ tile_counters, int M, int N, int K, int splits, int tiles_m, int tiles_n,
-               int n_units, int gated, int* status, const int* __restrict__ tile_group, int group_rows,
+               int n_units, FbGate gated, int* status, const int* __restrict__ tile_group, int group_rows,
                int plain_act) {
     // Grouped form (tile_group != nullptr): token tile t multiplies with the weight rows of group tile_group[t]
     // (rows [g * group_rows, g * group_rows + N) of the stacked matrix that map_w covers); a tile whose group is
@@ -249,10 +249,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
 #pragma unroll
                             for (int q = 0; q < 16; ++q) v[q] = 0.0f;
                         }
-                        if (gated) {
+                        if (gated.act) {
                             // output features alternate gate, up: even lanes hold a gate, their odd neighbour its
                             // up; the even lane writes act(gate) * up to column n / 2 of a half-as-wide output
-                            // (`gated` is the activation's code).
+                            // (`gated` is the activation with its constants).
                             // Every lane computes (straight-line code, sixteen independent chains); odd lanes'
                             // results are dropped.
                             float r[16];
@@ -355,7 +355,7 @@ int pick_splits(int tiles, int kb_total, int slots, int max_splits, double share
 template <int BN, typename TO, bool ACT = false>
 int launch_tc(const CUtensorMap& mw, const CUtensorMap& mx, void* out, long ldo, long slab_stride, int max_slabs,
               int* splits_used, float* partials, long partial_floats, int* counters, int n_counters, int M, int N,
-              int K, int force_splits, int* status, cudaStream_t stream, int gated = 0,
+              int K, int force_splits, int* status, cudaStream_t stream, FbGate gated = FbGate{0, 0.0f, 0.0f},
               const int* tile_group = nullptr, int group_rows = 0, int plain_act = 0) {
     using Cfg = TileCfg<BN>;
     const int tiles_n = (N + BM - 1) / BM, tiles_m = (M + BN - 1) / BN;
@@ -370,7 +370,7 @@ int launch_tc(const CUtensorMap& mw, const CUtensorMap& mx, void* out, long ldo,
                                        : 2.0 * BM * BN * BK / FB_MODEL_SM_FLOPS;
     const double share_cost_kb = ((double)M * N * 8.0 / FB_MODEL_HBM_BYTES_PER_S) / kb_seconds;
     int splits = force_splits > 0 ? force_splits : pick_splits(tiles, kb_total, slots, 16, share_cost_kb);
-    if (gated || tile_group) splits = 1;         // the activation needs the whole sum; grouped tiles are not split
+    if (gated.act || tile_group) splits = 1;         // the activation needs the whole sum; grouped tiles are not split
     if (splits > kb_total) splits = kb_total;
     if (slab_stride > 0) {
         if (splits > max_slabs) splits = max_slabs;
@@ -421,7 +421,7 @@ FB_API int fb_gemm_tc(const void* X, long long lda, const void* W, long long ldw
         if (const int shares = fb_gemm_pair_plan(M, N, K, slabs)) {
             if (splits_used) *splits_used = shares;
             return fb_launch_gemm_pair(X, (long)lda, W, (long)ldw, out, o_dtype, (long)ldo, (long)slab_stride, shares,
-                                       M, N, K, 0, 0, status, stream);
+                                       M, N, K, FbGate{0, 0.0f, 0.0f}, 0, status, stream);
         }
     }
     CUtensorMap mw, mx;
@@ -456,7 +456,7 @@ FB_API int fb_gemm_tc(const void* X, long long lda, const void* W, long long ldw
 // left as they are).  `act` is an FbPlainAct code.  For the products of routed experts over tokens sorted by expert.
 static int gemm_tc_grouped(const void* X, long long lda, const void* W, long long ldw, int groups,
                               const int* tile_group, int tile, void* out, int o_dtype, long long ldo, int M, int N,
-                              int K, int act, int gated, int* status, cudaStream_t stream) {
+                              int K, int act, FbGate gated, int* status, cudaStream_t stream) {
     FB_REQUIRE(M >= 0 && N > 0 && K > 0 && groups > 0, "gemm_tc_grouped: bad sizes M=%d N=%d K=%d", M, N, K);
     FB_REQUIRE(tile == 16 || tile == 32 || tile == 64 || tile == 128, "gemm_tc_grouped: row tiles of 16 to 128, not %d", tile);
     FB_REQUIRE(M % tile == 0 && tile_group, "gemm_tc_grouped: the rows must be whole tiles with a group each");
@@ -464,9 +464,9 @@ static int gemm_tc_grouped(const void* X, long long lda, const void* W, long lon
     FB_REQUIRE(lda % 8 == 0 && ldw % 8 == 0, "gemm_tc_grouped: row strides must be multiples of 8 elements");
     FB_REQUIRE(((uintptr_t)X & 15) == 0 && ((uintptr_t)W & 15) == 0, "gemm_tc_grouped: operands must be 16-byte aligned");
     FB_REQUIRE(fb_plain_act_known(act), "gemm_tc_grouped: unknown activation code %d", act);
-    FB_REQUIRE(!gated || (fb_act_known(gated) && !act && N % 2 == 0), "gemm_tc_grouped: a gate needs a known activation, "
+    FB_REQUIRE(!gated.act || (fb_gate_known(gated) && !act && N % 2 == 0), "gemm_tc_grouped: a gate needs a known activation, "
                "an even number of stacked rows and no plain activation beside it");
-    if (gated) FB_REQUIRE(ldo >= N / 2, "gemm_tc_grouped: a row stride is shorter than its row");
+    if (gated.act) FB_REQUIRE(ldo >= N / 2, "gemm_tc_grouped: a row stride is shorter than its row");
     else FB_REQUIRE(ldo >= N, "gemm_tc_grouped: a row stride is shorter than its row");
     FB_REQUIRE((long long)groups * N < 2147483647LL, "gemm_tc_grouped: too many weight rows");
     if (M == 0) return 0;
@@ -479,12 +479,12 @@ static int gemm_tc_grouped(const void* X, long long lda, const void* W, long lon
     case BN_:                                                                                                   \
         if (o_dtype == FB_F32)                                                                                  \
             return act ? launch_tc<BN_, float, true>(mw, mx, out, (long)ldo, 0, 1, nullptr, nullptr, 0, nullptr, 0, M, \
-                                                     N, K, 1, status, stream, 0, tile_group, N, act)            \
+                                                     N, K, 1, status, stream, FbGate{0, 0.0f, 0.0f}, tile_group, N, act)            \
                        : launch_tc<BN_, float>(mw, mx, out, (long)ldo, 0, 1, nullptr, nullptr, 0, nullptr, 0, M, N, K, \
                                                1, status, stream, gated, tile_group, N, 0);                         \
         else if (o_dtype == FB_BF16)                                                                            \
             return act ? launch_tc<BN_, __nv_bfloat16, true>(mw, mx, out, (long)ldo, 0, 1, nullptr, nullptr, 0, \
-                                                             nullptr, 0, M, N, K, 1, status, stream, 0,         \
+                                                             nullptr, 0, M, N, K, 1, status, stream, FbGate{0, 0.0f, 0.0f}, \
                                                              tile_group, N, act)                                \
                        : launch_tc<BN_, __nv_bfloat16>(mw, mx, out, (long)ldo, 0, 1, nullptr, nullptr, 0, nullptr, 0, \
                                                        M, N, K, 1, status, stream, gated, tile_group, N, 0);        \
@@ -502,15 +502,18 @@ static int gemm_tc_grouped(const void* X, long long lda, const void* W, long lon
 FB_API int fb_gemm_tc_grouped(const void* X, long long lda, const void* W, long long ldw, int groups,
                               const int* tile_group, int tile, void* out, int o_dtype, long long ldo, int M, int N,
                               int K, int act, int* status, cudaStream_t stream) {
-    return gemm_tc_grouped(X, lda, W, ldw, groups, tile_group, tile, out, o_dtype, ldo, M, N, K, act, 0, status, stream);
+    return gemm_tc_grouped(X, lda, W, ldw, groups, tile_group, tile, out, o_dtype, ldo, M, N, K, act, FbGate{0, 0.0f, 0.0f}, status, stream);
 }
 
 // The grouped form of the gated product: W [groups, N, K] stacks every group's gate and up rows alternately and
-// out[m, c] = act(g_c) * u_c with (g_0, u_0, g_1, u_1, ...) = X[m] * W[g]^T, `gated` an FbAct code; out has N / 2 columns.
+// out[m, c] = act(g_c) * u_c with (g_0, u_0, g_1, u_1, ...) = X[m] * W[g]^T, `act` an FbAct code with its constants; out
+// has N / 2 columns.
 FB_API int fb_gemm_tc_grouped_gated(const void* X, long long lda, const void* W, long long ldw, int groups,
                                     const int* tile_group, int tile, void* out, int o_dtype, long long ldo, int M,
-                                    int N, int K, int gated, int* status, cudaStream_t stream) {
-    FB_REQUIRE(fb_act_known(gated), "gemm_tc_grouped_gated: unknown activation code %d", gated);
+                                    int N, int K, int act, float limit, float slope, int* status,
+                                    cudaStream_t stream) {
+    const FbGate gated = {act, limit, slope};
+    FB_REQUIRE(fb_gate_known(gated), "gemm_tc_grouped_gated: unknown activation code %d, or its limit is not positive", act);
     return gemm_tc_grouped(X, lda, W, ldw, groups, tile_group, tile, out, o_dtype, ldo, M, N, K, 0, gated, status, stream);
 }
 
@@ -527,19 +530,21 @@ FB_API int fb_gemm_tc_add(const void* X, long long lda, const void* W, long long
     FB_REQUIRE(((uintptr_t)X & 15) == 0 && ((uintptr_t)W & 15) == 0, "gemm_tc_add: operands must be 16-byte aligned");
     if (M <= 128) return 0;
     if (fb_gemm_pair_plan(M, N, K, max_slabs < 1 ? 1 : max_slabs) != 1) return 0;
-    const int rc = fb_launch_gemm_pair(X, (long)lda, W, (long)ldw, acc, FB_F32, (long)ldacc, 0, 1, M, N, K, 0, 1, status,
-                                       stream);
+    const int rc = fb_launch_gemm_pair(X, (long)lda, W, (long)ldw, acc, FB_F32, (long)ldacc, 0, 1, M, N, K,
+                                       FbGate{0, 0.0f, 0.0f}, 1, status, stream);
     return rc ? rc : 1;
 }
 
 // out[M, N/2] = act(g) * u with [g_0, u_0, g_1, u_1, ...] = X[M,K] * W[N,K]^T: W stacks gate and up rows
-// alternately, and the activation `act` (an FbAct code) is applied in the epilogue (the whole sum in one CTA, so
+// alternately, and the activation `act_code` (an FbAct code with its constants) is applied in the epilogue (the whole sum in one CTA, so
 // K is not split).
 FB_API int fb_gemm_tc_gated(const void* X, long long lda, const void* W, long long ldw, void* out, int o_dtype,
-                            long long ldo, int M, int N, int K, int act, float* partials, long long partial_floats,
-                            int* counters, int n_counters, int* status, cudaStream_t stream) {
+                            long long ldo, int M, int N, int K, int act_code, float limit, float slope,
+                            float* partials, long long partial_floats, int* counters, int n_counters, int* status,
+                            cudaStream_t stream) {
+    const FbGate act = {act_code, limit, slope};
     FB_REQUIRE(M >= 0 && N > 0 && K > 0 && N % 2 == 0, "gemm_tc_gated: bad sizes M=%d N=%d K=%d", M, N, K);
-    FB_REQUIRE(fb_act_known(act), "gemm_tc_gated: unknown activation code %d", act);
+    FB_REQUIRE(fb_gate_known(act), "gemm_tc_gated: unknown activation code %d, or its limit is not positive", act_code);
     FB_REQUIRE(lda >= K && ldw >= K && ldo >= N / 2, "gemm_tc_gated: a row stride is shorter than its row");
     FB_REQUIRE(lda % 8 == 0 && ldw % 8 == 0, "gemm_tc_gated: row strides must be multiples of 8 elements");
     FB_REQUIRE(((uintptr_t)X & 15) == 0 && ((uintptr_t)W & 15) == 0, "gemm_tc_gated: operands must be 16-byte aligned");
@@ -594,10 +599,10 @@ FB_API int fb_gemm_tc_act(const void* X, long long lda, const void* W, long long
     case BN_:                                                                                                   \
         if (o_dtype == FB_F32)                                                                                  \
             return launch_tc<BN_, float, true>(mw, mx, out, (long)ldo, 0, 1, nullptr, nullptr, 0, nullptr, 0, M, N, K, \
-                                               1, status, stream, 0, nullptr, 0, act);                          \
+                                               1, status, stream, FbGate{0, 0.0f, 0.0f}, nullptr, 0, act);                          \
         else if (o_dtype == FB_BF16)                                                                            \
             return launch_tc<BN_, __nv_bfloat16, true>(mw, mx, out, (long)ldo, 0, 1, nullptr, nullptr, 0, nullptr, 0, \
-                                                       M, N, K, 1, status, stream, 0, nullptr, 0, act);         \
+                                                       M, N, K, 1, status, stream, FbGate{0, 0.0f, 0.0f}, nullptr, 0, act);         \
         break;
     switch (BN) {
         FB_TCA_CASE(16)

@@ -115,7 +115,7 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(P_THREADS, 1)
 gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                     const __grid_constant__ CUtensorMap map_o, int boxed_out,
                     TO* __restrict__ out, long ldo, long slab_stride, int M, int N, int K, int tiles_m, int tiles,
-                    int splits, int n_units, int gated, int accumulate, int* status) {
+                    int splits, int n_units, FbGate gated, int accumulate, int* status) {
     constexpr int S = P_STAGES;
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
@@ -259,7 +259,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                 // thread sends the box on its way (rows and columns beyond the output's edge are not written): a
                 // thousand 128-byte stores a tile from the warps themselves keep the epilogue waiting for the memory
                 // system's acknowledgements (7 us a tile against 2 to 3 us this way).
-                const int width = gated ? PBM / 2 : PBM;        // features of a staged row
+                const int width = gated.act ? PBM / 2 : PBM;        // features of a staged row
                 const bool leader = quarter == 0 && lane == 0;
 #pragma unroll 1
                 for (int c = half_id * 16; c < w.n_tok; c += 32) {
@@ -277,7 +277,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                         if (leader) bulk_wait_read();           // the box sent from this buffer, the one before last, has left it
                         asm volatile("bar.sync %0, 128;" ::"r"(2 + half_id) : "memory");
                     }
-                    if (gated) {
+                    if (gated.act) {
                         // features alternate gate, up: the even lane writes act(gate) * up to column n / 2
                         float r[16];
 #pragma unroll
@@ -312,7 +312,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
                         asm volatile("bar.sync %0, 128;" ::"r"(2 + half_id) : "memory");
                         if (leader) {
-                            const int x = (w.nt * (2 * PBM) + (int)rank * PBM) >> (gated ? 1 : 0);
+                            const int x = (w.nt * (2 * PBM) + (int)rank * PBM) >> (gated.act ? 1 : 0);
                             if (accumulate) tma_add_3d(&map_o, smem_u32(stage), x, m0 + c, w.split);
                             else tma_store_3d(&map_o, smem_u32(stage), x, m0 + c, w.split);
                             bulk_commit();
@@ -340,7 +340,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
 
 template <typename TO>
 int launch_pair(const void* X, long lda, const void* W, long ldw, void* out, long ldo, long slab_stride, int splits,
-                int M, int N, int K, int gated, int accumulate, int* status, cudaStream_t stream) {
+                int M, int N, int K, FbGate gated, int accumulate, int* status, cudaStream_t stream) {
     CUtensorMap mw, mx;
     int rc = fb_tensor_map_bf16(&mw, W, N, K, ldw, PBK, PBM);
     if (rc) return rc;
@@ -348,8 +348,8 @@ int launch_pair(const void* X, long lda, const void* W, long ldw, void* out, lon
     if (rc) return rc;
     // the output as boxes of 16 tokens x a CTA's features (half as many where the epilogue folds gate and up)
     CUtensorMap mo;
-    const int boxed = fb_tensor_map_out(&mo, out, (int)sizeof(TO), M, gated ? N / 2 : N, ldo, splits, slab_stride,
-                                        gated ? PBM / 2 : PBM, P_OUT_TOKENS);
+    const int boxed = fb_tensor_map_out(&mo, out, (int)sizeof(TO), M, gated.act ? N / 2 : N, ldo, splits, slab_stride,
+                                        gated.act ? PBM / 2 : PBM, P_OUT_TOKENS);
     if (boxed < 0) return boxed;
     auto kern = gemm_tc_pair_kernel<TO>;
     static bool configured[FB_MAX_DEVICES] = {};
@@ -405,11 +405,11 @@ int fb_gemm_pair_plan(int M, int N, int K, int max_slabs) {
 }
 
 int fb_launch_gemm_pair(const void* X, long lda, const void* W, long ldw, void* out, int o_dtype, long ldo,
-                        long slab_stride, int splits, int M, int N, int K, int gated, int accumulate, int* status,
+                        long slab_stride, int splits, int M, int N, int K, FbGate gated, int accumulate, int* status,
                         cudaStream_t stream) {
-    if (splits < 1 || (splits > 1 && (slab_stride <= 0 || o_dtype != FB_F32 || gated)))
+    if (splits < 1 || (splits > 1 && (slab_stride <= 0 || o_dtype != FB_F32 || gated.act)))
         return fb_fail(-1, "gemm_tc_pair: %d shares of K need float32 slabs", splits);
-    if (accumulate && (o_dtype != FB_F32 || splits != 1 || gated))
+    if (accumulate && (o_dtype != FB_F32 || splits != 1 || gated.act))
         return fb_fail(-1, "gemm_tc_pair: only a whole float32 product can be added to its output");
     if (o_dtype == FB_F32)
         return launch_pair<float>(X, lda, W, ldw, out, ldo, slab_stride, splits, M, N, K, gated, accumulate, status,

@@ -8,7 +8,10 @@
 //                logits over all experts, the `top` largest of score + bias are chosen, the weights are the chosen
 //                scores themselves, divided by their sum and multiplied by `weight_scale`.  A third rule (`rule` 2):
 //                scores = sigmoid of every logit by itself, the `top` largest of score + bias are chosen, the weights
-//                are the chosen scores as they are, times `weight_scale`
+//                are the chosen scores as they are, times `weight_scale`.  The rules with scores may keep the weights as
+//                they are or divide them by their sum (`renorm`), and may choose within groups: the experts form equal
+//                groups of neighbours, a group counts as its largest score + bias, and only experts of the best
+//                `keep_groups` groups (the lower one on a tie) can be chosen
 //   moe_sort     one CTA: (token, choice) pairs counted per expert, every expert's stretch padded to a multiple of
 //                the products' row tile, so that a row tile belongs to one expert; writes for every place of the
 //                padded order its token (-1: padding), for every pair its place, for every row tile its expert
@@ -23,7 +26,8 @@ template <typename TW>
 __global__ void __launch_bounds__(128)
 moe_choose_kernel(const float* __restrict__ z_in, long z_stride, int n_partials, long partial_stride,
                   const TW* __restrict__ br, int gate_col, int n, int E, int K, int* __restrict__ chosen,
-                  float* __restrict__ share, float* __restrict__ gate, int rule, float weight_scale) {
+                  float* __restrict__ share, float* __restrict__ gate, int rule, float weight_scale, int renorm,
+                  int group_size, int keep_groups) {
     fb_pdl_launch_dependents();
     fb_pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -63,6 +67,31 @@ moe_choose_kernel(const float* __restrict__ z_in, long z_stride, int n_partials,
             const int e = lane + 32 * r;
             z[r] = e < E ? s[r] + (br ? fb_to_float(br[e]) : 0.0f) : -INFINITY;
         }
+        if (keep_groups > 0) {
+            // the groups one after another, the best first: the largest number among the experts whose group is not
+            // in yet names the next group; what is in no kept group cannot be chosen
+            unsigned in = 0;                           // bit r: the group of this lane's expert lane + 32 r is in
+            for (int k = 0; k < keep_groups; ++k) {
+                float best = -INFINITY;
+                int best_e = 0x7fffffff;
+#pragma unroll
+                for (int r = 0; r < MOE_MAX_LOGITS_PER_LANE; ++r)
+                    if (!(in >> r & 1u) && z[r] > best) { best = z[r]; best_e = lane + 32 * r; }
+#pragma unroll
+                for (int off = 16; off > 0; off >>= 1) {
+                    const float ob = __shfl_xor_sync(0xffffffffu, best, off);
+                    const int oe = __shfl_xor_sync(0xffffffffu, best_e, off);
+                    if (ob > best || (ob == best && oe < best_e)) { best = ob; best_e = oe; }
+                }
+                const int group = best_e / group_size;
+#pragma unroll
+                for (int r = 0; r < MOE_MAX_LOGITS_PER_LANE; ++r)
+                    if ((lane + 32 * r) / group_size == group) in |= 1u << r;
+            }
+#pragma unroll
+            for (int r = 0; r < MOE_MAX_LOGITS_PER_LANE; ++r)
+                if (!(in >> r & 1u)) z[r] = -INFINITY;
+        }
         float total = 0.0f, mine = 0.0f;               // lane k keeps the k-th chosen score
         for (int k = 0; k < K; ++k) {
             float best = -INFINITY, best_s = 0.0f;
@@ -86,7 +115,7 @@ moe_choose_kernel(const float* __restrict__ z_in, long z_stride, int n_partials,
             if (lane == k) mine = best_s;
             if (lane == 0) chosen[(size_t)row * K + k] = best_e;
         }
-        if (lane < K) share[(size_t)row * K + lane] = (rule == 1 ? mine / (total + 1e-20f) : mine) * weight_scale;
+        if (lane < K) share[(size_t)row * K + lane] = (renorm ? mine / (total + 1e-20f) : mine) * weight_scale;
         if (gate_col >= 0 && lane == 0) gate[row] = 1.0f / (1.0f + expf(-logit(gate_col)));
         return;
     }
@@ -253,24 +282,28 @@ FB_API int fb_moe_gather_rows(const void* h, long long h_stride, int dtype, cons
 }
 
 // rule 0: the `top` largest logits + bias, weights = softmax over the chosen; rule 1: scores = softmax over all E, the
-// `top` largest of score + bias, weights = chosen scores / their sum * weight_scale; rule 2: scores = sigmoid of each
-// logit, the `top` largest of score + bias, weights = chosen scores * weight_scale.
+// `top` largest of score + bias, weights = chosen scores * weight_scale; rule 2: scores = sigmoid of each logit, the rest
+// as in rule 1.  Rules 1 and 2: renorm divides the chosen scores by their sum; keep_groups > 0 chooses within the best
+// that many of n_groups equal groups of neighbouring experts.
 // z: float32 router logits [n, >= E (+1)] (possibly split-K shares), as a product of the token rows with the stacked
 // router matrix left them; br: the router's bias or nullptr; gate_col: the column that holds w_gate . h (negative: none).
 FB_API int fb_moe_choose(const float* z, long long z_stride, int n_partials, long long partial_stride, const void* br,
                          int w_dtype, int gate_col, int n, int E, int K, int* chosen, float* share, float* gate,
-                         int rule, float weight_scale, cudaStream_t stream) {
+                         int rule, float weight_scale, int renorm, int n_groups, int keep_groups, cudaStream_t stream) {
     FB_REQUIRE(rule >= 0 && rule <= 2, "router: unknown rule %d", rule);
     FB_REQUIRE(n >= 0 && E > 0 && K > 0 && K <= E, "router: bad sizes n=%d experts=%d top=%d", n, E, K);
     FB_REQUIRE(E <= 32 * MOE_MAX_LOGITS_PER_LANE, "router: %d experts are more than %d", E, 32 * MOE_MAX_LOGITS_PER_LANE);
     FB_REQUIRE(K <= 32, "router: top = %d is more than 32", K);
+    FB_REQUIRE(n_groups >= 1 && E % n_groups == 0, "router: %d experts do not form %d equal groups", E, n_groups);
+    FB_REQUIRE(keep_groups >= 0 && keep_groups <= n_groups && (keep_groups == 0 || (rule != 0 && K <= keep_groups * (E / n_groups))),
+               "router: %d experts cannot be chosen from %d groups of %d", K, keep_groups, E / n_groups);
     FB_REQUIRE(gate_col < 0 || gate, "router: a gate column without a place for the gate");
     FB_REQUIRE(z_stride >= E && z_stride > gate_col, "router: logit rows are too short");
     if (n == 0) return 0;
     if (n_partials < 1) n_partials = 1;
     FB_DISPATCH_DTYPE(w_dtype, TW,
         (fb_launch((moe_choose_kernel<TW>), dim3((n + 3) / 4), dim3(128), 0, stream, z, (long)z_stride, n_partials,
-                   (long)partial_stride, (const TW*)br, gate_col, n, E, K, chosen, share, gate, rule, weight_scale)));
+                   (long)partial_stride, (const TW*)br, gate_col, n, E, K, chosen, share, gate, rule, weight_scale, renorm, E / n_groups, keep_groups)));
     return fb_check_launch("moe_choose");
 }
 

@@ -6,8 +6,13 @@
 // that size shared by the heads) or over the whole projection at once (FB_QK_NORM_PROJECTION: width = heads * head
 // size, a weight of that size), before the rotation in both cases.  The weight enters as (w + weight_offset).
 // Rotation: the first 2 * half dimensions of a head, dimension i paired with i + half, angles from the step's
-// cos/sin tables [n, half]; the rest of the head passes unchanged.  Value rows have a width of their own.
-#include "common.cuh"
+// cos/sin tables [n, half]; the rest of the head passes unchanged.  Value rows have a width of their own, and their
+// columns may be the keys' (`v_off`): the values are then the keys as projected, before norm and rotation.
+//
+// Heads that are normalised alone (or not at all) and whose sizes are multiples of 4 go to a second kernel, one warp a
+// head: shares fetched 16 bytes at a time, the norm within the warp, the pairs exchanged through the warp's own stretch
+// of shared memory.
+#include "rows.cuh"
 
 enum FbQkNorm : int { FB_QK_NORM_NONE = 0, FB_QK_NORM_HEAD = 1, FB_QK_NORM_PROJECTION = 2 };
 
@@ -26,7 +31,7 @@ qk_norm_rope_kv_write_kernel(const float* __restrict__ proj, long proj_stride, i
                              const int* __restrict__ row_seq, const int* __restrict__ block_table, int table_stride,
                              const int* __restrict__ table_base, int table_head, T* __restrict__ k_pool,
                              T* __restrict__ v_pool, int page_size, int n_pages, int nh, int nkv, int hd, int vd,
-                             int write_kv, int* status) {
+                             int v_off, int write_kv, int* status) {
     fb_pdl_launch_dependents();
     fb_pdl_wait();
     extern __shared__ float sh[];                      // [qw + kw] the row's q and k; then one factor per head
@@ -107,12 +112,112 @@ qk_norm_rope_kv_write_kernel(const float* __restrict__ proj, long proj_stride, i
         for (int e = tid; e < vw; e += blockDim.x) {
             const int g = e / vd, d = e - g * vd;
             v_dst[(size_t)g * page_size * vd + d] =
-                fb_from_float<T>(qkr_slab_sum(pr, qw + kw + e, n_partials, partial_stride));
+                fb_from_float<T>(qkr_slab_sum(pr, v_off + e, n_partials, partial_stride));
         }
     }
 }
 
-// proj: float32 rows [q: nh*hd | k: nkv*hd | v: nkv*vd], possibly as n_partials shares partial_stride elements apart.
+// One warp per (row, head): heads 0 .. nh - 1 are queries, the nkv behind them keys, the nkv behind those values (none
+// where the values are the keys as projected: the key's warp then writes both).  NV = float4 a lane holds of a head.
+constexpr int QKR_WARPS = 8;
+template <typename TW, typename T, int NV>
+__global__ void __launch_bounds__(32 * QKR_WARPS)
+qk_norm_rope_heads_kernel(const float* __restrict__ proj, long proj_stride, int n_partials, long partial_stride,
+                          const TW* __restrict__ q_weight, const TW* __restrict__ k_weight, float eps,
+                          float weight_offset, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
+                          int half, T* __restrict__ q_out, long q_out_stride, const int* __restrict__ positions,
+                          const int* __restrict__ row_seq, const int* __restrict__ block_table, int table_stride,
+                          const int* __restrict__ table_base, int table_head, T* __restrict__ k_pool,
+                          T* __restrict__ v_pool, int page_size, int n_pages, int n, int nh, int nkv, int hd, int vd,
+                          int v_off, int v_is_k, int write_kv, int* status) {
+    fb_pdl_launch_dependents();
+    fb_pdl_wait();
+    extern __shared__ float sh[];                      // [QKR_WARPS][hd]
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int per_row = nh + (write_kv ? (v_is_k ? nkv : 2 * nkv) : 0);
+    const long item = (long)blockIdx.x * QKR_WARPS + warp;
+    if (item >= (long)n * per_row) return;
+    const int row = (int)(item / per_row), h = (int)(item - (long)row * per_row);
+    const bool is_q = h < nh, is_v = h >= nh + nkv;
+    const int g = is_q ? h : is_v ? h - nh - nkv : h - nh;
+    const int width = is_v ? vd : hd, nvec = width >> 2;
+    const float* src = proj + (size_t)row * proj_stride + (is_q ? (size_t)h * hd : is_v ? (size_t)v_off + (size_t)g * vd
+                                                                                        : (size_t)(nh + g) * hd);
+    float4 x[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = lane + 32 * i;
+        x[i] = c < nvec ? slab_sum4(src + 4 * c, n_partials, partial_stride) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    T* k_dst = nullptr;
+    T* v_dst = nullptr;
+    if (!is_q) {
+        const int p = positions[row], seq = row_seq[row];
+        const int entry = fb_table_column(p / page_size, table_base ? table_base[seq] : 0, table_head);
+        const int page = (entry >= 0 && entry < table_stride) ? block_table[(size_t)seq * table_stride + entry] : -1;
+        if (page < 0 || page >= n_pages) {
+            if (lane == 0) atomicOr(status, FB_STATUS_BAD_PAGE);
+            return;
+        }
+        const size_t at = ((size_t)page * nkv + g) * page_size + (p % page_size);
+        k_dst = k_pool + at * hd;
+        v_dst = v_pool + at * vd;
+    }
+    if (is_v || (!is_q && v_is_k)) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int c = lane + 32 * i;
+            if (c < nvec) Vec4<T>::store(v_dst + 4 * c, x[i]);
+        }
+        if (is_v) return;
+    }
+    const TW* w = is_q ? q_weight : k_weight;
+    if (w) {
+        float s = 0.0f;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) s += x[i].x * x[i].x + x[i].y * x[i].y + x[i].z * x[i].z + x[i].w * x[i].w;
+        const float f = 1.0f / sqrtf(fb_warp_sum(s) / (float)hd + eps);
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int c = lane + 32 * i;
+            if (c >= nvec) continue;
+            const float4 wv = Vec4<TW>::load(w + 4 * c);
+            x[i].x *= f * (wv.x + weight_offset); x[i].y *= f * (wv.y + weight_offset);
+            x[i].z *= f * (wv.z + weight_offset); x[i].w *= f * (wv.w + weight_offset);
+        }
+    }
+    if (half > 0) {
+        float* mine = sh + (size_t)warp * hd;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int c = lane + 32 * i;
+            if (4 * c < 2 * half) Vec4<float>::store(mine + 4 * c, x[i]);
+        }
+        __syncwarp();
+        const float* cs = cos_t + (size_t)row * half;
+        const float* sn = sin_t + (size_t)row * half;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int d0 = 4 * (lane + 32 * i);
+            if (d0 >= 2 * half) continue;
+            float* xe = reinterpret_cast<float*>(&x[i]);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int d = d0 + e;
+                if (d < half) xe[e] = xe[e] * cs[d] - mine[d + half] * sn[d];
+                else if (d < 2 * half) xe[e] = xe[e] * cs[d - half] + mine[d - half] * sn[d - half];
+            }
+        }
+    }
+    T* dst = is_q ? q_out + (size_t)row * q_out_stride + (size_t)h * hd : k_dst;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = lane + 32 * i;
+        if (c < nvec) Vec4<T>::store(dst + 4 * c, x[i]);
+    }
+}
+
+// proj: float32 rows [q: nh*hd | k: nkv*hd | ... v: nkv*vd from column v_off on ...], possibly as n_partials shares partial_stride elements apart.
 // q_weight / k_weight (dtype w_dtype): [hd] each for FB_QK_NORM_HEAD, [nh*hd] and [nkv*hd] for FB_QK_NORM_PROJECTION.
 FB_API int fb_qk_norm_rope_kv_write(const float* proj, long long proj_stride, int n_partials, long long partial_stride,
                                     const void* q_weight, const void* k_weight, int w_dtype, int scope, float eps,
@@ -120,17 +225,45 @@ FB_API int fb_qk_norm_rope_kv_write(const float* proj, long long proj_stride, in
                                     long long q_out_stride, int out_dtype, const int* positions, const int* row_seq,
                                     const int* block_table, int table_stride, const int* table_base, int table_head,
                                     void* k_pool, void* v_pool, int page_size, int n_pages, int n, int nh, int nkv, int hd, int vd,
-                                    int write_kv, int* status, cudaStream_t stream) {
+                                    int v_off, int write_kv, int* status, cudaStream_t stream) {
     FB_REQUIRE(n >= 0 && nh > 0 && nkv > 0 && hd > 0 && vd > 0, "qk_norm_rope_kv_write: bad sizes");
     FB_REQUIRE(scope >= FB_QK_NORM_NONE && scope <= FB_QK_NORM_PROJECTION, "qk_norm_rope_kv_write: unknown reach %d", scope);
     FB_REQUIRE(half >= 0 && 2 * half <= hd, "qk_norm_rope_kv_write: rotary width %d exceeds head size %d", 2 * half, hd);
     FB_REQUIRE(half == 0 || (cos_t && sin_t), "qk_norm_rope_kv_write: rotary tables missing");
     FB_REQUIRE(!write_kv || (positions && row_seq && block_table && k_pool && v_pool && page_size > 0 && n_pages > 0),
                "qk_norm_rope_kv_write: cache arguments missing");
-    FB_REQUIRE(proj_stride >= (long long)nh * hd + (long long)nkv * hd + (long long)nkv * vd,
+    const int k_off = nh * hd;
+    FB_REQUIRE(v_off >= k_off && (v_off != k_off || vd == hd), "qk_norm_rope_kv_write: values that are the keys have their size");
+    FB_REQUIRE(proj_stride >= (long long)(nh + nkv) * hd && proj_stride >= (long long)v_off + (long long)nkv * vd,
                "qk_norm_rope_kv_write: projection rows are too short");
     if (n == 0) return 0;
     if (n_partials < 1) n_partials = 1;
+    const size_t esize = out_dtype == FB_BF16 ? 2 : 4;
+    const size_t wsize = w_dtype == FB_BF16 ? 2 : 4;
+    auto aligned = [](const void* p, size_t to) { return (uintptr_t)p % to == 0; };
+    if (scope != FB_QK_NORM_PROJECTION && hd % 4 == 0 && vd % 4 == 0 && hd <= 512 && vd <= 512 && v_off % 4 == 0 &&
+        proj_stride % 4 == 0 && partial_stride % 4 == 0 && q_out_stride % 4 == 0 && aligned(proj, 16) &&
+        aligned(q_out, 4 * esize) && aligned(k_pool, 4 * esize) && aligned(v_pool, 4 * esize) &&
+        aligned(q_weight, 4 * wsize) && aligned(k_weight, 4 * wsize)) {
+        if (scope == FB_QK_NORM_NONE) q_weight = k_weight = nullptr;
+        const int v_is_k = v_off == k_off ? 1 : 0;
+        const long items = (long)n * (nh + (write_kv ? (v_is_k ? nkv : 2 * nkv) : 0));
+        const unsigned blocks = (unsigned)((items + QKR_WARPS - 1) / QKR_WARPS);
+        const size_t smem_h = (size_t)QKR_WARPS * hd * sizeof(float);
+        const int widest = hd > vd ? hd : vd;
+#define FB_QKR_HEADS(NV_)                                                                                             \
+        FB_DISPATCH_DTYPE(w_dtype, TW, FB_DISPATCH_DTYPE(out_dtype, T,                                                \
+            (fb_launch((qk_norm_rope_heads_kernel<TW, T, NV_>), dim3(blocks), dim3(32 * QKR_WARPS), smem_h, stream, proj, \
+                       (long)proj_stride, n_partials, (long)partial_stride, (const TW*)q_weight, (const TW*)k_weight, eps, \
+                       weight_offset, cos_t, sin_t, half, (T*)q_out, (long)q_out_stride, positions, row_seq, block_table, \
+                       table_stride, table_base, table_head, (T*)k_pool, (T*)v_pool, page_size, n_pages, n, nh, nkv, hd, vd, \
+                       v_off, v_is_k, write_kv, status))))
+        if (widest <= 128) FB_QKR_HEADS(1);
+        else if (widest <= 256) FB_QKR_HEADS(2);
+        else FB_QKR_HEADS(4);
+#undef FB_QKR_HEADS
+        return fb_check_launch("qk_norm_rope_kv_write");
+    }
     const size_t smem = ((size_t)(nh + nkv) * hd + nh + nkv) * sizeof(float);
     FB_REQUIRE(smem <= 200 * 1024, "qk_norm_rope_kv_write: a row of q and k (%zu bytes) does not fit shared memory", smem);
     FB_DISPATCH_DTYPE(w_dtype, TW, FB_DISPATCH_DTYPE(out_dtype, T, {
@@ -140,7 +273,7 @@ FB_API int fb_qk_norm_rope_kv_write(const float* proj, long long proj_stride, in
         fb_launch(kernel, dim3(n), dim3(n > 128 ? 256 : cols >= 4096 ? 1024 : cols >= 1024 ? 512 : 256), smem, stream, proj, (long)proj_stride, n_partials, (long)partial_stride,
                   (const TW*)q_weight, (const TW*)k_weight, scope, eps, weight_offset, cos_t, sin_t, half, (T*)q_out,
                   (long)q_out_stride, positions, row_seq, block_table, table_stride, table_base, table_head, (T*)k_pool,
-                  (T*)v_pool, page_size, n_pages, nh, nkv, hd, vd, write_kv, status);
+                  (T*)v_pool, page_size, n_pages, nh, nkv, hd, vd, v_off, write_kv, status);
     }));
     return fb_check_launch("qk_norm_rope_kv_write");
 }

@@ -32,11 +32,14 @@ _SIGNATURES = {
     "fb_add_rmsnorm": (I, [P, P, I, I, L, P, I, P, I, P, I, I, F, F, STREAM]),
     "fb_rope_table": (I, [P, P, P, P, I, I, F, STREAM]),
     "fb_rope_kv_write": (I, [P, L, I, L, P, L, P, L, P, L, I, I, P, P, I, P, P, P, I, P, I, P, P, I, I, I, I, I, I, I, P, STREAM]),
-    "fb_gate_mul": (I, [P, L, I, I, L, P, I, I, I, I, STREAM]),
+    "fb_gate_mul": (I, [P, L, I, I, L, P, I, I, I, I, F, F, STREAM]),
     "fb_activation": (I, [P, L, I, I, L, P, I, I, I, I, STREAM]),
-    "fb_add_row": (I, [P, P, I, I, I, STREAM]),
-    "fb_add_slabs": (I, [P, P, I, L, I, I, STREAM]),
+    "fb_add_row": (I, [P, P, P, I, I, I, STREAM]),
+    "fb_add_slabs": (I, [P, P, I, L, P, I, I, I, STREAM]),
     "fb_sigmoid_gate": (I, [P, L, I, P, L, I, L, I, I, STREAM]),
+    # token_inputs.cu
+    "fb_embedding_pairs": (I, [P, P, I, P, P, P, P, P, P, L, L, L, I, P, I, I, I, F, P, STREAM]),
+    "fb_token_gate": (I, [P, L, I, L, P, I, L, I, P, I, P, I, I, I, I, P, STREAM]),
     # hyper_connections.cu
     "fb_hc_step": (I, [P, L, I, P, I, L, P, P, P, P, I, F, F, P, I, P, I, I, I, STREAM]),
     "fb_branch_norm_mix": (I, [I, P, P, P, P, I, P, F, F, P, I, I, STREAM]),
@@ -47,20 +50,20 @@ _SIGNATURES = {
     "fb_gemm_tc_add": (I, [P, L, P, L, P, L, I, I, I, I, P, STREAM]),
     "fb_gemm_tc": (I, [P, L, P, L, P, I, L, L, I, P, I, I, I, P, L, P, I, I, P, STREAM]),
     "fb_gemm_tc_grouped": (I, [P, L, P, L, I, P, I, P, I, L, I, I, I, I, P, STREAM]),
-    "fb_gemm_tc_grouped_gated": (I, [P, L, P, L, I, P, I, P, I, L, I, I, I, I, P, STREAM]),
+    "fb_gemm_tc_grouped_gated": (I, [P, L, P, L, I, P, I, P, I, L, I, I, I, I, F, F, P, STREAM]),
     "fb_gemm_tc_act": (I, [P, L, P, L, P, I, L, I, I, I, I, P, STREAM]),
-    "fb_gemm_tc_gated": (I, [P, L, P, L, P, I, L, I, I, I, I, P, L, P, I, P, STREAM]),
+    "fb_gemm_tc_gated": (I, [P, L, P, L, P, I, L, I, I, I, I, F, F, P, L, P, I, P, STREAM]),
     # attention_simt.cu
-    "fb_paged_attention_simt": (I, [P, L, P, L, I, P, P, I, I, P, I, P, I, P, P, I, I, I, I, I, I, I, F, P, P, P, STREAM]),
+    "fb_paged_attention_simt": (I, [P, L, P, L, I, P, P, I, I, P, I, P, I, P, P, I, I, I, I, I, I, I, F, F, P, P, P, L, I, L, P, STREAM]),
     # qk_norm_rope.cu
     "fb_qk_norm_rope_kv_write": (I, [P, L, I, L, P, P, I, I, F, F, P, P, I, P, L, I, P, P, P, I, P, I, P, P, I, I, I, I,
-                                     I, I, I, I, P, STREAM]),
+                                     I, I, I, I, I, P, STREAM]),
     # gated_delta.cu
     "fb_gdr_prepare": (I, [P, L, I, L, P, I, P, P, I, P, L, L, P, P, P, P, I, P, P, P, I, I, I, I, I, F, F, STREAM]),
     "fb_gdr_recurrent": (I, [P, P, P, P, L, P, P, P, I, P, I, I, I, I, STREAM]),
     "fb_gdr_out_norm": (I, [P, P, L, I, L, I, P, I, F, P, I, I, I, I, STREAM]),
     # moe.cu
-    "fb_moe_choose": (I, [P, L, I, L, P, I, I, I, I, I, P, P, P, I, F, STREAM]),
+    "fb_moe_choose": (I, [P, L, I, L, P, I, I, I, I, I, P, P, P, I, F, I, I, I, STREAM]),
     "fb_moe_max_tiles": (I, [I, I, I]),
     "fb_moe_gather_rows": (I, [P, L, I, P, P, I, I, P, P, STREAM]),
     "fb_moe_sort": (I, [P, I, I, I, I, I, P, P, P, P, STREAM]),
@@ -88,8 +91,8 @@ _SIGNATURES = {
     "fb_diff_attention_mma": (I, [P, L, P, L, P, P, P, I, I, P, I, P, P, P, P, I, I, I, I, I, I, I, I, I, F, F, F, F, I,
                                   P, L, P, STREAM]),
     # attention_mma.cu
-    "fb_paged_attention_mma": (I, [P, L, P, L, P, P, I, I, P, I, P, I, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, P, P, I,
-                                   P, L, P, L, L, I, P, STREAM]),
+    "fb_paged_attention_mma": (I, [P, L, P, L, P, P, I, I, P, I, P, I, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, F, P, P,
+                                   P, L, I, L, I, P, L, P, L, L, I, P, STREAM]),
     # sampling.cu
     "fb_apply_penalties": (I, [P, L, I, P, P, P, P, P, P, I, STREAM]),
     "fb_apply_logit_bias": (I, [P, L, I, P, P, P, I, STREAM]),

@@ -8,6 +8,7 @@ from __future__ import annotations
 
 import ctypes
 import os
+from dataclasses import dataclass
 
 import torch
 
@@ -242,18 +243,31 @@ def rope_kv_write(q_in, q_out, k, v, cos, sin, half: int, positions, row_seq, bl
         _stream()), "rope_kv_write")
 
 
-ACTIVATIONS = {"silu": 1, "gelu_tanh": 2, "gelu_pytorch_tanh": 2}      # codes of the kernels' gate activations
+ACTIVATIONS = {"silu": 1, "gelu_tanh": 2, "gelu_pytorch_tanh": 2, "limited": 3}   # codes of the kernels' gate activations
 
 
-def activation_code(name: str) -> int:
-    try:
-        return ACTIVATIONS[name]
-    except KeyError:
-        raise KernelError(f"activation '{name}' is not implemented; known: {', '.join(sorted(ACTIVATIONS))}") from None
+@dataclass(frozen=True)
+class GateActivation:
+    """An activation of gated feed-forwards with its constants.  'limited': with g = min(gate, limit) and u = up held
+    to [-limit, limit], the result is g sigmoid(slope g) (u + 1); the other names have no constants, and may stand as
+    plain strings wherever this class is taken."""
+    name: str
+    limit: float = 0.0
+    slope: float = 1.0
+
+
+def gate_arguments(activation) -> tuple:
+    """(code, limit, slope) of a gate activation: a name of ACTIVATIONS or a GateActivation."""
+    a = activation if isinstance(activation, GateActivation) else GateActivation(activation)
+    if a.name not in ACTIVATIONS:
+        raise KernelError(f"activation '{a.name}' is not implemented; known: {', '.join(sorted(ACTIVATIONS))}")
+    if a.name == "limited" and not a.limit > 0.0:
+        raise KernelError(f"activation 'limited' needs a positive limit, not {a.limit}")
+    return ACTIVATIONS[a.name], float(a.limit), float(a.slope)
 
 
 def gate_mul(gate_up: torch.Tensor, out: torch.Tensor, n_partials: int = 1, partial_stride: int = 0,
-             activation: str = "silu") -> None:
+             activation="silu") -> None:
     """out[:, c] = act(gate_up[:, 2c]) * gate_up[:, 2c+1] (gate and up alternate along a row); with
     n_partials > 1, gate_up is the first of that many split-K shares `partial_stride` elements apart, which are
     added first."""
@@ -263,7 +277,7 @@ def gate_mul(gate_up: torch.Tensor, out: torch.Tensor, n_partials: int = 1, part
     if tuple(out.shape) != (n, I) or not out.is_contiguous():
         raise KernelError("gate_mul: bad output")
     check(lib().fb_gate_mul(gate_up.data_ptr(), _rows(gate_up), dtype_code(gate_up), int(n_partials),
-                            int(partial_stride), out.data_ptr(), dtype_code(out), n, I, activation_code(activation),
+                            int(partial_stride), out.data_ptr(), dtype_code(out), n, I, *gate_arguments(activation),
                             _stream()), "gate_mul")
 
 
@@ -292,23 +306,66 @@ def activation(z: torch.Tensor, out: torch.Tensor, name: str, n_partials: int = 
           "activation")
 
 
-def add_row(x: torch.Tensor, v: torch.Tensor) -> None:
-    """x[r] += v for every row of the contiguous float32 x."""
-    _cuda(x, v)
+def add_row(x: torch.Tensor, v, y=None) -> None:
+    """x[r] += y[r] + v for every row of the contiguous float32 x; v (a vector) or y (float32 rows) may be None."""
+    _cuda(x, v, y)
     n, H = x.shape
-    if x.dtype != torch.float32 or not x.is_contiguous() or v.numel() != H or not v.is_contiguous():
+    if x.dtype != torch.float32 or not x.is_contiguous() or (v is not None and (v.numel() != H or not v.is_contiguous())):
         raise KernelError("add_row: a contiguous float32 [n, H] and a vector of H wanted")
-    check(lib().fb_add_row(x.data_ptr(), v.data_ptr(), dtype_code(v), n, H, _stream()), "add_row")
+    if y is not None and (y.dtype != torch.float32 or tuple(y.shape) != (n, H) or not y.is_contiguous()):
+        raise KernelError("add_row: the rows to add must be contiguous float32 like x")
+    check(lib().fb_add_row(x.data_ptr(), _ptr(y), _ptr(v), dtype_code(v) if v is not None else 0, n, H, _stream()),
+          "add_row")
 
 
-def add_slabs(x: torch.Tensor, delta: torch.Tensor, n: int, n_partials: int = 1, partial_stride: int = 0) -> None:
-    """x[:n] += delta[:n] (and the further shares of delta, `partial_stride` elements apart); contiguous float32."""
-    _cuda(x, delta)
-    if x.dtype != torch.float32 or delta.dtype != torch.float32 or not x.is_contiguous() or not delta.is_contiguous() \
-            or x.shape[1] != delta.shape[-1]:
+def add_slabs(x: torch.Tensor, delta, n: int, n_partials: int = 1, partial_stride: int = 0, copy=None) -> None:
+    """x[:n] += delta[:n] (and the further shares of delta, `partial_stride` elements apart); contiguous float32.
+    copy (optional, [n, H] in either dtype): receives the rows of x as they then are; delta may then be None (nothing
+    to add)."""
+    _cuda(x, delta, copy)
+    if x.dtype != torch.float32 or not x.is_contiguous() or x.shape[0] < n or \
+            (delta is not None and (delta.dtype != torch.float32 or not delta.is_contiguous()
+                                    or x.shape[1] != delta.shape[-1])):
         raise KernelError("add_slabs: contiguous float32 rows of one width wanted")
-    check(lib().fb_add_slabs(x.data_ptr(), delta.data_ptr(), int(n_partials), int(partial_stride), int(n), x.shape[1],
-                             _stream()), "add_slabs")
+    if copy is not None and (copy.shape[0] < n or copy.shape[1] != x.shape[1] or not copy.is_contiguous()):
+        raise KernelError("add_slabs: the copy must be contiguous rows of the stream's width")
+    check(lib().fb_add_slabs(x.data_ptr(), _ptr(delta), int(n_partials), int(partial_stride), _ptr(copy),
+                             dtype_code(copy) if copy is not None else 0, int(n), x.shape[1], _stream()), "add_slabs")
+
+
+def embedding_pairs(table: torch.Tensor, pairs: torch.Tensor, mul_prev: int, mul_cur: int, ids: torch.Tensor, batch,
+                    state: torch.Tensor, x: torch.Tensor, status: torch.Tensor, scale: float = 1.0) -> None:
+    """x[t] = table[ids[t]] * scale + pairs[row], row = (mul_prev * id before + mul_cur * ids[t]) mod buckets, or the
+    last row of `pairs` [buckets + 1, H] for a request's first token.  state: int32 [slots, 1], the id of the last
+    token of every request + 1 (0: none yet); read for an entry's first token and updated."""
+    _cuda(table, pairs, ids, state, x, status)
+    _i32(ids, "token ids")
+    _i32(state, "state")
+    V, H = table.shape
+    n, buckets = ids.numel(), pairs.shape[0] - 1
+    if x.dtype != torch.float32 or x.shape[0] < n or x.shape[1] != H or not x.is_contiguous() or pairs.dtype != table.dtype \
+            or pairs.shape[1] != H or buckets < 1 or not table.is_contiguous() or not pairs.is_contiguous():
+        raise KernelError("embedding_pairs: a contiguous float32 stream and two tables of its width in one dtype wanted")
+    check(lib().fb_embedding_pairs(
+        table.data_ptr(), pairs.data_ptr(), dtype_code(table), ids.data_ptr(), batch.row_seq.data_ptr(),
+        batch.seq_q_start_d.data_ptr(), batch.seq_q_len_d.data_ptr(), batch.seq_slot_d.data_ptr(), state.data_ptr(),
+        state.stride(0), int(mul_prev) % buckets, int(mul_cur) % buckets, buckets, x.data_ptr(), n, H, V, float(scale),
+        status.data_ptr(), _stream()), "embedding_pairs")
+
+
+def token_gate(z: torch.Tensor, table: torch.Tensor, offset: int, dim: int, ids: torch.Tensor, out: torch.Tensor,
+               status: torch.Tensor, n_partials: int = 1, partial_stride: int = 0) -> None:
+    """out[t, c] = gelu(z[t, c]) * table[ids[t], offset + c] for c < dim, 0 behind it; z float32 [n, >= dim], possibly
+    the first of n_partials shares."""
+    _cuda(z, table, ids, out, status)
+    _i32(ids, "token ids")
+    n, cols = out.shape
+    if z.dtype != torch.float32 or z.shape[0] < n or not out.is_contiguous() or table.stride(1) != 1 or ids.numel() < n:
+        raise KernelError("token_gate: bad shapes")
+    check(lib().fb_token_gate(z.data_ptr(), _rows(z), int(n_partials), int(partial_stride), table.data_ptr(),
+                              dtype_code(table), table.stride(0), int(offset), ids.data_ptr(), table.shape[0],
+                              out.data_ptr(), dtype_code(out), n, int(dim), cols, status.data_ptr(), _stream()),
+          "token_gate")
 
 
 def branch_norm_mix(branches, eps: float, out: torch.Tensor, n: int, weight_offset: float = 0.0) -> None:
@@ -374,14 +431,28 @@ def _slopes(score_slopes, nh: int) -> int:
     return score_slopes.data_ptr()
 
 
+def _head_gate(head_gate, n: int, nh: int) -> tuple:
+    """(address, row stride, shares, stride of the shares) of a gate per head: head_gate = (float32 view [n, nh] whose
+    rows may lie apart, how many shares, their stride), or None for none."""
+    if head_gate is None:
+        return 0, 0, 1, 0
+    g, parts, stride = head_gate
+    _cuda(g)
+    if g.dtype != torch.float32 or g.shape[0] < n or g.shape[1] != nh:
+        raise KernelError("attention: a gate per head is one float32 per row and query head")
+    return g.data_ptr(), _rows(g), int(parts), int(stride)
+
+
 def paged_attention_simt(q, out, k_pool, v_pool, block_table, positions, row_seq, nh: int, nkv: int, hd: int,
                          window: int, scale: float, status, table_base=None, score_slopes=None, sinks=None,
-                         vd: int = 0, keep_first: int = 0, table_head: int = 0) -> None:
+                         vd: int = 0, keep_first: int = 0, table_head: int = 0, softcap: float = 0.0,
+                         head_gate=None) -> None:
     """score_slopes (float32 per query head, optional): slope * (key position - query position) is added to every
     scaled score, a linear penalty on distance.  sinks (float32 per query head, optional): one more softmax slot per
     head whose score is that number, unscaled, and which has no value.  vd: the size of a value row where it is not
     the key row's (the output then has nh * vd columns).  keep_first: under a window, the keys at positions below
-    this stay visible to every later query."""
+    this stay visible to every later query.  softcap > 0: scores are softcap * tanh(scale * q.k / softcap).  head_gate
+    (see _head_gate): every head's output is multiplied by sigmoid of its number."""
     _cuda(q, out, k_pool, v_pool, block_table, positions, row_seq, status, table_base, sinks)
     _i32(table_base, "table_base")
     n = q.shape[0]
@@ -399,8 +470,9 @@ def paged_attention_simt(q, out, k_pool, v_pool, block_table, positions, row_seq
     check(lib().fb_paged_attention_simt(
         q.data_ptr(), _rows(q), out.data_ptr(), _rows(out), dtype_code(q), k_pool.data_ptr(), v_pool.data_ptr(),
         page_size, n_pages, block_table.data_ptr(), block_table.stride(0), _ptr(table_base), int(table_head),
-        positions.data_ptr(), row_seq.data_ptr(), n, nh, nkv, hd, vd, int(window), int(keep_first), float(scale), _slopes(score_slopes, nh),
-        _ptr(sinks), status.data_ptr(), _stream()), "paged_attention_simt")
+        positions.data_ptr(), row_seq.data_ptr(), n, nh, nkv, hd, vd, int(window), int(keep_first), float(scale), float(softcap),
+        _slopes(score_slopes, nh), _ptr(sinks), *_head_gate(head_gate, n, nh), status.data_ptr(), _stream()),
+        "paged_attention_simt")
 
 
 def apply_penalties(logits, rows, tokens, counts, repetition, presence, frequency) -> None:
@@ -508,7 +580,7 @@ def gemm_tc_add(a: torch.Tensor, w: torch.Tensor, acc: torch.Tensor, status: tor
 
 
 def gemm_tc_gated(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, status: torch.Tensor,
-                  activation: str = "silu") -> None:
+                  activation="silu") -> None:
     """out[M, N/2] = act(g) * u where (g_0, u_0, g_1, u_1, ...) = a @ w^T: w stacks gate and up rows alternately
     and the activation runs in the product's epilogue."""
     _cuda(a, w, out, status)
@@ -518,7 +590,7 @@ def gemm_tc_gated(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, status: t
         raise KernelError(f"gated gemm: shapes a{tuple(a.shape)} w{tuple(w.shape)} out{tuple(out.shape)} do not agree")
     partials, counters = _SplitScratch.get(a.device)
     check(lib().fb_gemm_tc_gated(a.data_ptr(), _rows(a), w.data_ptr(), _rows(w), out.data_ptr(), dtype_code(out),
-                                 _rows(out), M, N, K, activation_code(activation), partials.data_ptr(),
+                                 _rows(out), M, N, K, *gate_arguments(activation), partials.data_ptr(),
                                  partials.numel(), counters.data_ptr(), counters.numel(), status.data_ptr(),
                                  _stream()), "gemm_tc_gated", (M, N, K))
 
@@ -598,7 +670,7 @@ def gemm_tc_grouped(a: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor, 
 
 
 def gemm_tc_grouped_gated(a: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor, tile: int, out: torch.Tensor,
-                          status: torch.Tensor, activation: str) -> None:
+                          status: torch.Tensor, activation) -> None:
     """out[m, c] = act(g_c) * u_c with (g_0, u_0, g_1, u_1, ...) = a[m] @ w[tile_group[m // tile]]^T on the tcgen05
     kernel: w [groups, 2 I, K] stacks every group's gate and up rows alternately, out has I columns."""
     _cuda(a, w, tile_group, out, status)
@@ -609,12 +681,12 @@ def gemm_tc_grouped_gated(a: torch.Tensor, w: torch.Tensor, tile_group: torch.Te
         raise KernelError("grouped gated gemm: shapes do not agree")
     check(lib().fb_gemm_tc_grouped_gated(a.data_ptr(), _rows(a), w.data_ptr(), K, groups, tile_group.data_ptr(),
                                          int(tile), out.data_ptr(), dtype_code(out), _rows(out), M, N, K,
-                                         activation_code(activation), status.data_ptr(), _stream()),
+                                         *gate_arguments(activation), status.data_ptr(), _stream()),
           "gemm_tc_grouped_gated", (M, N, K))
 
 
 def grouped_gated_linear(a: torch.Tensor, row_index, w: torch.Tensor, tile_group: torch.Tensor, tile: int,
-                         out: torch.Tensor, activation: str, ctx, row_share=None, row_pair=None) -> None:
+                         out: torch.Tensor, activation, ctx, row_share=None, row_pair=None) -> None:
     """out[m] = act(gate) * up of a[row_index[m]] under the weights of the row tile's group (w [groups, 2 I, K], gate
     and up rows alternating): on the tcgen05 kernel with the activation in its epilogue for bfloat16 operands, else
     the float32-FMA grouped product followed by the activation kernel.  row_share / row_pair (with row_index): the
@@ -737,7 +809,8 @@ def paged_attention_mma(q, out, k_pool, v_pool, block_table, seq_q_start, seq_q_
                         max_q_len: int, max_kv_len: int, any_short: bool, any_long: bool, nh: int, nkv: int,
                         hd: int, window: int, scale: float, status, table_base=None, prefetch=None,
                         multi_seqs=None, n_multi: int = 0, score_slopes=None, sinks=None,
-                        weights_float32: bool = False, keep_first: int = 0, table_head: int = 0) -> None:
+                        weights_float32: bool = False, keep_first: int = 0, table_head: int = 0,
+                        softcap: float = 0.0, head_gate=None) -> None:
     """bfloat16 attention on the tensor cores over the paged cache; sequences are described per entry of the
     step (first row, rows, first position).  any_short / any_long say whether the step holds sequences with
     rows * (nh/nkv) <= 16 / > 16 (attention_is_short), which run in different arrangements of the kernel.  table_base (int32 per
@@ -751,7 +824,8 @@ def paged_attention_mma(q, out, k_pool, v_pool, block_table, seq_q_start, seq_q_
     rounding left: 16 bits of mantissa, two MMAs for one) instead of rounded to bfloat16; portions then run on the
     mma.sync kernel, whose weights are in registers.  keep_first: under a window, the keys at positions below this
     stay visible to every later query (their tiles are walked ahead of the window's; portions then run on the
-    mma.sync kernel)."""
+    mma.sync kernel).  softcap > 0: scores are softcap * tanh(scale * q.k / softcap); head_gate (see _head_gate): every
+    head's output is multiplied by sigmoid of its number (portions run on the mma.sync kernel with either)."""
     _cuda(q, out, k_pool, v_pool, block_table, seq_q_start, seq_q_len, seq_pos_start, status, table_base, multi_seqs,
           sinks)
     if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != nh or not sinks.is_contiguous()):
@@ -771,8 +845,8 @@ def paged_attention_mma(q, out, k_pool, v_pool, block_table, seq_q_start, seq_q_
         block_table.data_ptr(), block_table.stride(0), _ptr(table_base), int(table_head), seq_q_start.data_ptr(),
         seq_q_len.data_ptr(), seq_pos_start.data_ptr(), _ptr(multi_seqs), int(n_multi), n_seqs, max_q_len, max_kv_len,
         1 if any_short else 0,
-        1 if any_long else 0, nh, nkv, hd, int(window), int(keep_first), float(scale), _slopes(score_slopes, nh), _ptr(sinks),
-        1 if weights_float32 else 0, scratch.data_ptr(), scratch.numel(),
+        1 if any_long else 0, nh, nkv, hd, int(window), int(keep_first), float(scale), float(softcap),
+        _slopes(score_slopes, nh), _ptr(sinks), *_head_gate(head_gate, q.shape[0], nh), 1 if weights_float32 else 0, scratch.data_ptr(), scratch.numel(),
         *prefetch_arguments(prefetch), status.data_ptr(), _stream()), "paged_attention_mma", (n_seqs, nkv, hd))
 
 
@@ -793,7 +867,7 @@ def attention_is_short(q_len: int, nh: int, nkv: int) -> bool:
 
 def paged_attention(ctx, q, out, cache, nh: int, nkv: int, hd: int, window: int, scale: float,
                     next_weight=None, score_slopes=None, sinks=None, vd: int = 0, weights_float32: bool = False,
-                    keep_first: int = 0) -> None:
+                    keep_first: int = 0, softcap: float = 0.0, head_gate=None) -> None:
     """Attention of every row of the step over its request's cached keys: the tensor-core kernel for bfloat16
     and head sizes it takes, the float32 CUDA-core kernel otherwise (all of the 32-bit mode).  next_weight: the
     matrix of the product that follows, whose start the bfloat16 kernel may fetch into L2 (a hint)."""
@@ -806,12 +880,13 @@ def paged_attention(ctx, q, out, cache, nh: int, nkv: int, hd: int, window: int,
                             nh, nkv, hd, window, scale, ctx.runtime.status, table_base=cache.table_base,
                             prefetch=next_weight, multi_seqs=b.multi_seqs_d, n_multi=b.n_multi,
                             score_slopes=score_slopes, sinks=sinks, weights_float32=weights_float32,
-                            keep_first=keep_first, table_head=cache.table_head)
+                            keep_first=keep_first, table_head=cache.table_head, softcap=softcap,
+                            head_gate=head_gate)
     else:
         paged_attention_simt(q, out, cache.k_pool, cache.v_pool, cache.block_table, b.positions, b.row_seq,
                              nh, nkv, hd, window, scale, ctx.runtime.status, table_base=cache.table_base,
                              score_slopes=score_slopes, sinks=sinks, vd=vd, keep_first=keep_first,
-                             table_head=cache.table_head)
+                             table_head=cache.table_head, softcap=softcap, head_gate=head_gate)
 
 
 def diff_attention_mma_supported(q: torch.Tensor, nh: int, nkv: int, kd: int, vd: int) -> bool:
@@ -895,8 +970,9 @@ QK_NORM_REACH = {None: 0, "none": 0, "head": 1, "projection": 2}
 
 def qk_norm_rope_kv_write(proj: torch.Tensor, q_weight, k_weight, reach, eps: float, weight_offset: float, cos, sin,
                           half: int, q_out: torch.Tensor, cache, positions, row_seq, nh: int, nkv: int, hd: int,
-                          vd: int, status, n_partials: int = 1, partial_stride: int = 0) -> None:
-    """proj: float32 rows [q: nh*hd | k: nkv*hd | v: nkv*vd] (possibly split-K shares).  q and k pass an RMS norm
+                          vd: int, status, n_partials: int = 1, partial_stride: int = 0, v_off: int | None = None) -> None:
+    """proj: float32 rows [q: nh*hd | k: nkv*hd | v: nkv*vd] (possibly split-K shares; v_off: the column the values
+    begin at where that is not right behind the keys; the keys' own first column: the values are the keys as projected).  q and k pass an RMS norm
     whose reach is a head ('head': weights [hd]) or the whole projection ('projection': weights [nh*hd] and
     [nkv*hd]) or none, then the rotation of the first 2*half dimensions of every head (cos/sin float32 [n, half]);
     q goes to q_out in its dtype, k and v into the cache's pages when the view is writable."""
@@ -921,6 +997,7 @@ def qk_norm_rope_kv_write(proj: torch.Tensor, q_weight, k_weight, reach, eps: fl
         _ptr(sin), int(half), q_out.data_ptr(), _rows(q_out), dtype_code(q_out), positions.data_ptr(),
         row_seq.data_ptr(), cache.block_table.data_ptr(), cache.block_table.stride(0), _ptr(cache.table_base),
         int(cache.table_head), k_pool.data_ptr(), v_pool.data_ptr(), cache.page_size, n_pages, n, nh, nkv, hd, vd,
+        (nh + nkv) * hd if v_off is None else int(v_off),
         1 if cache.writable else 0, status.data_ptr(), _stream()), "qk_norm_rope_kv_write")
 
 
@@ -983,12 +1060,18 @@ ROUTER_RULES = {"softmax_of_chosen": 0, "softmax_of_all": 1, "sigmoid": 2}
 
 
 def moe_choose(z, bias, gate_col: int, experts: int, top: int, chosen, share, gate, n_partials: int = 1,
-               partial_stride: int = 0, rule: str = "softmax_of_chosen", weight_scale: float = 1.0) -> None:
+               partial_stride: int = 0, rule: str = "softmax_of_chosen", weight_scale: float = 1.0,
+               renormalize=None, groups: int = 1, keep_groups: int = 0) -> None:
     """Per token: the `top` experts with the largest logits z[:, :experts] + bias (float32; z possibly split-K
     shares), their softmax weights, and (gate_col >= 0) gate = sigmoid(z[:, gate_col]).  rule 'softmax_of_all':
     scores = softmax(z) over all experts, the `top` largest of score + bias are chosen, and the weights are the chosen
     scores over their sum, times `weight_scale`.  rule 'sigmoid': scores = sigmoid of every logit by itself, the `top`
-    largest of score + bias are chosen, and the weights are the chosen scores as they are, times `weight_scale`."""
+    largest of score + bias are chosen, and the weights are the chosen scores as they are, times `weight_scale`.
+    renormalize (None: as the rule says): whether those two rules divide the chosen scores by their sum.
+    keep_groups > 0: they choose among the experts of the best that many of `groups` equal groups of neighbours, a
+    group counting as its largest score + bias."""
+    if renormalize is None:
+        renormalize = rule == "softmax_of_all"
     if rule not in ROUTER_RULES:
         raise KernelError(f"router: rule '{rule}' is not one of {sorted(ROUTER_RULES)}")
     _cuda(z, bias, chosen, share, gate)
@@ -999,7 +1082,8 @@ def moe_choose(z, bias, gate_col: int, experts: int, top: int, chosen, share, ga
     check(lib().fb_moe_choose(z.data_ptr(), _rows(z), int(n_partials), int(partial_stride), _ptr(bias),
                               dtype_code(bias) if bias is not None else 0, int(gate_col), n, int(experts), int(top),
                               chosen.data_ptr(), share.data_ptr(), _ptr(gate), ROUTER_RULES[rule],
-                              float(weight_scale), _stream()), "moe_choose")
+                              float(weight_scale), 1 if renormalize else 0, int(groups), int(keep_groups), _stream()),
+          "moe_choose")
 
 
 def moe_max_tiles(pairs: int, experts: int, tile: int) -> int:

@@ -41,6 +41,16 @@ class DecoderModel:
                 specs[name] = ts
         return specs
 
+    def shared_tensor_names(self) -> set:
+        """Tensors that more than one part wants (a table of which every layer reads its own columns): they are kept on
+        the device once."""
+        seen, shared = set(), set()
+        for p in self.parts():
+            names = set(p.tensor_specs())
+            shared |= seen & names
+            seen |= names
+        return shared
+
     def bind(self, tensors: dict) -> None:
         for p in self.parts():
             p.bind(tensors)
@@ -66,7 +76,14 @@ class DecoderModel:
             # (a block that keeps state beside its mixer's, such as the inputs a convolution still needs, says so)
             state = block.state_requirement() if hasattr(block, "state_requirement") else mixer.state_requirement()
             plans.append(CallPlan(kv=mixer.cache_requirement(), state=state, cache_from=call.cache_from))
+        # an embedding that keeps something per request (the token before, say) has an entry behind the layer calls
+        state = self._embedding_state()
+        if state is not None:
+            plans.append(CallPlan(state=state))
         return plans
+
+    def _embedding_state(self):
+        return self.embedding.state_requirement() if hasattr(self.embedding, "state_requirement") else None
 
     # ---- one step -------------------------------------------------------------
     def forward(self, ctx) -> torch.Tensor | None:
@@ -74,7 +91,10 @@ class DecoderModel:
         rt, b = self.runtime, ctx.batch
         n = b.n_tokens
         x = ctx.open_stream(self.hidden_size)
-        self.embedding.forward(ctx, b.token_ids[:n], x)
+        if self._embedding_state() is not None:
+            self.embedding.forward(ctx, b.token_ids[:n], x, state=ctx.cache(len(self.order)).state)
+        else:
+            self.embedding.forward(ctx, b.token_ids[:n], x)
         stream = ResidualStream(x)
         x0 = None
         if self.reentry is not None:

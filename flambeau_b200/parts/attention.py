@@ -44,9 +44,13 @@ class PagedAttention(Mixer):
     `keep_first` (with a window): the keys at positions below this stay visible to every later query, each with the
     position it was written at (which its rotation and the window's distances use); the pages that hold them are kept
     while the request lives, whatever the window gives back behind them.
-    `gate` (bool): the heads' outputs are multiplied element by element by sigmoid(Wg h) before the output projection
-    (`<prefix><names.g>`, [num_heads * value_dim, width]; Wg reads the same input as the other projections and is
-    part of their one product).
+    `gate`: sigmoid(Wg h) multiplies the heads' outputs before the output projection; Wg (`<prefix><names.g>`) reads the
+    same input as the other projections and is part of their one product.  True (or 'element'): element by element,
+    Wg [num_heads * value_dim, width], a kernel of its own behind the attention; 'head': one number per head,
+    Wg [num_heads, width], applied where the attention kernels write a head's output.
+    `softcap` (> 0): every scaled score passes cap * tanh(score / cap) before the softmax (float32).
+    `values_from_keys`: there is no Wv; the values are the keys as projected, before norm and rotation (their size is
+    the keys').
     `names`: what the tensors are called behind the prefix (keys q, k, v, o, q_norm, k_norm, sink, g), for checkpoints
     with other names than the defaults."""
     graph_safe = True
@@ -58,11 +62,20 @@ class PagedAttention(Mixer):
                  window: int = 0, position: PartSpec | None = None, scale: float | None = None,
                  init_std: float = 0.02, qk_norm: PartSpec | None = None, distance_slopes=None,
                  qk_norm_reach: str = "head", value_dim: int | None = None, sink: bool = False, names=None,
-                 weights_float32: bool = False, keep_first: int = 0, gate: bool = False):
+                 weights_float32: bool = False, keep_first: int = 0, gate=False, softcap: float = 0.0,
+                 values_from_keys: bool = False):
         super().__init__(runtime, prefix)
-        self.gate = bool(gate)
+        if gate not in (False, True, None, "element", "head"):
+            raise ValueError(f"attention: gate = {gate!r}: 'element', 'head' or none")
+        self.gate = {True: "element", False: None}.get(gate, gate)
+        self.softcap = float(softcap or 0.0)
+        if self.softcap < 0.0:
+            raise ValueError(f"attention: softcap = {softcap} must be positive (0 or None: none)")
+        self.values_from_keys = bool(values_from_keys)
         self.width, self.nh, self.nkv, self.hd = int(width), int(num_heads), int(num_kv_heads), int(head_dim)
         self.vd = int(value_dim) if value_dim else self.hd
+        if self.values_from_keys and self.vd != self.hd:
+            raise ValueError(f"attention: values that are the keys are as wide as they are ({self.vd} against {self.hd})")
         self.sink = bool(sink)
         self.weights_float32 = bool(weights_float32)
         self.names = dict(self.DEFAULT_NAMES)
@@ -114,23 +127,25 @@ class PagedAttention(Mixer):
         specs = {
             p + nm["q"]: TensorSpec((self.qw, self.width), init=init),
             p + nm["k"]: TensorSpec((self.kvw, self.width), init=init),
-            p + nm["v"]: TensorSpec((self.vw, self.width), init=init),
             p + nm["o"]: TensorSpec((self.width, self.nh * self.vd), init=init),
         }
+        if not self.values_from_keys:
+            specs[p + nm["v"]] = TensorSpec((self.vw, self.width), init=init)
         if self.sink:
             specs[p + nm["sink"]] = TensorSpec((self.nh,), init=("normal", 1.0))
         if self.gate:
-            specs[p + nm["g"]] = TensorSpec((self.nh * self.vd, self.width), init=init)
+            specs[p + nm["g"]] = TensorSpec((self.nh * self.vd if self.gate == "element" else self.nh, self.width),
+                                            init=init)
         return specs
 
     def own_bind(self, tensors):
         p, nm = self.prefix, self.names
-        stack = [tensors[p + nm["q"]], tensors[p + nm["k"]], tensors[p + nm["v"]]]
+        stack = [tensors[p + nm[name]] for name in (("q", "k") if self.values_from_keys else ("q", "k", "v"))]
         self.gate_off = sum(t.shape[0] for t in stack)          # the gate's columns lie behind q, k and v
         if self.gate:
             stack.append(tensors[p + nm["g"]])
         rows = sum(t.shape[0] for t in stack)
-        if rows % 8 and (self.q_norm is not None or self.vd != self.hd) and self._fused_norm_kernel():
+        if rows % 8 and (self._wants_norm_kernel() or self.gate == "head") and self._fused_norm_kernel():
             # rows of zeros up to a multiple of 8, so that the product's float32 rows stay 16-byte aligned
             stack.append(torch.zeros((8 - rows % 8, self.width), dtype=stack[0].dtype, device=stack[0].device))
         self.qkv = Linear(concat_rows(stack))
@@ -141,6 +156,11 @@ class PagedAttention(Mixer):
     def own_weights(self):
         return [self.qkv.weight, self.o.weight]
 
+    def _wants_norm_kernel(self) -> bool:
+        """Whether the mixer needs what only the kernel of _fused_norm_kernel does: a norm of q and k, values of their
+        own width, or values that are the keys as projected."""
+        return self.q_norm is not None or self.vd != self.hd or self.values_from_keys
+
     def _fused_norm_kernel(self) -> bool:
         """Whether the kernel that normalises, rotates and writes the cache in one pass serves this mixer: the norms
         (if any) are the framework's RMS norm and the position encoding hands out its tables."""
@@ -149,6 +169,12 @@ class PagedAttention(Mixer):
         if pos is not None and not getattr(pos, "fused_with_cache_write", False):
             return False
         return all(n is None or type(n) is RMSNorm for n in (self.q_norm, self.k_norm))
+
+    def _head_gate(self, slabs, parts):
+        """What the attention kernels want of a gate per head: its columns of the product, as shares."""
+        if self.gate != "head":
+            return None
+        return slabs[0][:, self.gate_off:self.gate_off + self.nh], parts, slabs.stride(0)
 
     def forward(self, ctx, h, out, call):
         n = ctx.n_tokens
@@ -160,7 +186,7 @@ class PagedAttention(Mixer):
             fused = pos is None or getattr(pos, "fused_with_cache_write", False)
             # the fused rotary kernel adds split-K shares of the projection itself; a position encoding with a
             # rotate() of its own gets whole rows
-            if (self.q_norm is not None or self.vd != self.hd) and self._fused_norm_kernel():
+            if self._wants_norm_kernel() and self._fused_norm_kernel():
                 # one product for q, k and v; one kernel adds its shares, normalises q and k (every head alone or
                 # the whole projection at once), rotates them, rounds q and fills the cache's pages
                 cols = self.qkv.out_features
@@ -174,19 +200,21 @@ class PagedAttention(Mixer):
                     self.k_norm.weight if qn is not None else None, self.qk_norm_reach if qn is not None else None,
                     qn.eps if qn is not None else 0.0, qn.weight_offset if qn is not None else 0.0, cos, sin,
                     pos.half if pos is not None else 0, q, cache, ctx.batch.positions, ctx.batch.row_seq, self.nh,
-                    self.nkv, self.hd, self.vd, rt.status, n_partials=parts, partial_stride=slabs.stride(0))
+                    self.nkv, self.hd, self.vd, rt.status, n_partials=parts, partial_stride=slabs.stride(0),
+                    v_off=self.qw if self.values_from_keys else None)
                 a = ctx.ws.alloc((n, self.nh * self.vd), rt.dtype)
                 hint = self.o.weight if ctx.l2_hints and n <= 64 else None
                 ops.paged_attention(ctx, q, a, cache, self.nh, self.nkv, self.hd, self.window, self.scale,
                                     next_weight=hint, score_slopes=self.distance_slopes, sinks=self.sinks, vd=self.vd,
-                                    weights_float32=self.weights_float32, keep_first=self.keep_first)
-                if self.gate:
+                                    weights_float32=self.weights_float32, keep_first=self.keep_first,
+                                    softcap=self.softcap, head_gate=self._head_gate(slabs, parts))
+                if self.gate == "element":
                     ops.sigmoid_gate(a, slabs[0][:, self.gate_off:self.gate_off + self.nh * self.vd], n, parts,
                                      slabs.stride(0))
                 ctx.to_stream(self.o, a)
                 return
-            if self.vd != self.hd or self.qk_norm_reach != "head":
-                raise ValueError("attention: value rows of their own width, or a norm over the whole projection, "
+            if self.vd != self.hd or self.values_from_keys or self.qk_norm_reach != "head":
+                raise ValueError("attention: value rows of their own width, or from the keys, or a norm over the whole projection, "
                                  "need the framework's RMS norm and a position encoding that hands out its tables")
             if self.gate and self.q_norm is not None:
                 raise ValueError("attention: an output gate beside query/key norms needs the framework's RMS norm and a "
@@ -232,8 +260,9 @@ class PagedAttention(Mixer):
             hint = self.o.weight if ctx.l2_hints and n <= 64 else None
             ops.paged_attention(ctx, q, a, cache, self.nh, self.nkv, self.hd, self.window, self.scale,
                                 next_weight=hint, score_slopes=self.distance_slopes, sinks=self.sinks,
-                                weights_float32=self.weights_float32, keep_first=self.keep_first)
-            if self.gate:
+                                weights_float32=self.weights_float32, keep_first=self.keep_first, softcap=self.softcap,
+                                head_gate=self._head_gate(qkv_slabs, parts) if self.gate else None)
+            if self.gate == "element":
                 ops.sigmoid_gate(a, qkv_slabs[0][:, self.gate_off:self.gate_off + self.qw], n, parts, stride)
             ctx.to_stream(self.o, a)
 

@@ -24,7 +24,8 @@ Categories and the method each must have:
                  where the block keeps state of its own beside its mixer's.
   input_map      forward(ctx, h, out, state, offset): what a sublayer reads, made from the normalised rows h
                  (float32) into `out` (engine dtype); state_floats(): float32 numbers it keeps per request.
-  embedding      forward(ctx, token_ids, x).
+  embedding      forward(ctx, token_ids, x); optionally state_requirement() where it keeps something per request, and
+                 then forward(ctx, token_ids, x, state=...).
   head           forward(ctx, h_rows, logits).
 
 `ctx` is an engine.step.StepContext: the batch descriptor on the device, the

@@ -5,6 +5,7 @@ import torch
 
 from ..kernels import ops
 from .base import Part, StateRequirement, TensorSpec
+from .linear import Linear
 from .spec import PartSpec, build_part, register_part
 
 
@@ -120,6 +121,130 @@ class PreNormBlock(Part):
             self.feed_forward.forward(ctx, h, delta)
             stream.pending, stream.pending_slabs = delta, ctx.pending_slabs
         ctx.stream_x = None                   # another kind of block decides for itself whether parts may add to its stream
+
+
+class ParallelBlock(Part):
+    """x <- x + (mixer(h) + feed_forward(h)) with h = norm(x): one norm, whose rows both sublayers read.
+    `feed_forward` may be None.  The two outputs stay pending together: the feed-forward's float32 shares lie right
+    behind the mixer's, so that whoever adds what is pending adds one run of shares; over a portion a sublayer's last
+    product may add to the stream by itself, which nothing reads again before the next norm."""
+    graph_safe = True
+    category = "block"
+    SLABS = "parallel.slabs"
+
+    def __init__(self, runtime=None, prefix="", *, mixer: PartSpec, norm: PartSpec, feed_forward: PartSpec | None = None):
+        super().__init__(runtime, prefix)
+        self.mixer = build_part(mixer, runtime)
+        self.norm = build_part(norm, runtime)
+        self.feed_forward = build_part(feed_forward, runtime) if feed_forward is not None else None
+
+    def children(self):
+        return [p for p in (self.norm, self.mixer, self.feed_forward) if p is not None]
+
+    def forward(self, ctx, stream: ResidualStream, call) -> None:
+        h = ctx.normed
+        ctx.stream_x = stream.x
+        self.norm.add_norm(ctx, stream.x, stream.pending, h, n_partials=stream.pending_slabs,
+                           delta_norm=stream.pending_norm)
+        stream.pending_norm = None
+        slabs = ctx.shared.get(self.SLABS)
+        if slabs is None:                     # room for both sublayers' shares, the step's own for one of them
+            slabs = ctx.shared[self.SLABS] = ctx.step_alloc((2 * ctx.max_slabs, *ctx.delta.shape), torch.float32)
+        kept = (ctx.delta_slabs, ctx.delta)
+        used = 0
+        try:
+            for part in (self.mixer, self.feed_forward):
+                if part is None:
+                    continue
+                mine = slabs[used:used + ctx.max_slabs]
+                ctx.delta_slabs, ctx.delta, ctx.pending_slabs = mine, mine[0], 1
+                if part is self.mixer:
+                    part.forward(ctx, h, mine[0], call)
+                else:
+                    part.forward(ctx, h, mine[0])
+                used += ctx.pending_slabs     # (0: the part has added its output to the stream)
+        finally:
+            ctx.delta_slabs, ctx.delta = kept
+        stream.pending, stream.pending_slabs = slabs[0], used
+        ctx.stream_x = None
+
+
+class TokenInputBlock(Part):
+    """A block behind which every token's id gives the stream something of its own: with x the stream after the inner
+    block and e the layer's `dim` columns (from `offset` on) of the token's row in a table that all layers share,
+
+        x <- x + norm(Wproj (gelu(Wgate x) * e))
+
+    (gelu in its tanh form; Wgate [dim, width] and Wproj [width, dim] read and write the stream without a norm in front).
+    The result stays pending with its norm, which the next norm's kernel applies while it adds.  Tensors:
+    `<prefix><names.gate>`, `<prefix><names.proj>`, the norm's own, and the table `table` [vocab, table_width]."""
+    graph_safe = True
+    category = "block"
+
+    def __init__(self, runtime=None, prefix="", *, block: PartSpec, norm: PartSpec, width: int, dim: int, offset: int,
+                 vocab: int, table: str, table_width: int, names=None, init_std: float = 0.02):
+        super().__init__(runtime, prefix)
+        self.inner = build_part(block, runtime)
+        self.norm = build_part(norm, runtime)
+        self.width, self.dim, self.offset, self.vocab = int(width), int(dim), int(offset), int(vocab)
+        self.table_name, self.table_width, self.init_std = table, int(table_width), init_std
+        if self.dim < 1 or not 0 <= self.offset <= self.table_width - self.dim:
+            raise ValueError(f"token input: columns [{offset}, {offset + dim}) of a table with {table_width}")
+        self.names = dict({"gate": "gate", "proj": "proj"}, **(names or {}))
+        self.cols = -(-self.dim // 8) * 8      # columns of zeros up to a multiple of 8, for the products' alignment
+        self.gate = self.proj = self.table = None
+
+    @property
+    def mixer(self):
+        return self.inner.mixer
+
+    @property
+    def feed_forward(self):
+        return self.inner.feed_forward
+
+    def state_requirement(self):
+        inner = self.inner
+        return inner.state_requirement() if hasattr(inner, "state_requirement") else inner.mixer.state_requirement()
+
+    def children(self):
+        return [self.inner, self.norm]
+
+    def own_tensor_specs(self):
+        p, init = self.prefix, ("normal", self.init_std)
+        return {p + self.names["gate"]: TensorSpec((self.dim, self.width), init=init),
+                p + self.names["proj"]: TensorSpec((self.width, self.dim), init=init),
+                self.table_name: TensorSpec((self.vocab, self.table_width), init=("normal", 1.0))}
+
+    def own_bind(self, tensors):
+        gate, proj = tensors[self.prefix + self.names["gate"]], tensors[self.prefix + self.names["proj"]]
+        pad = self.cols - self.dim
+        self.gate = Linear(torch.nn.functional.pad(gate, (0, 0, 0, pad)).contiguous())
+        self.proj = Linear(torch.nn.functional.pad(proj, (0, pad)).contiguous())
+        self.table = tensors[self.table_name]
+
+    def own_weights(self):
+        return [self.gate.weight, self.proj.weight]       # (a step reads n rows of the table, not the table)
+
+    def forward(self, ctx, stream: ResidualStream, call) -> None:
+        self.inner.forward(ctx, stream, call)
+        n = ctx.n_tokens
+        if stream.pending_norm is not None:
+            stream.settle(ctx)
+        with ctx.ws.scope():
+            rows = stream.x[:n]
+            pending = stream.pending if stream.pending_slabs > 0 else None
+            if self.runtime.dtype != torch.float32:        # the product's operand, as the stream with all of it added
+                rows = ctx.ws.alloc((n, self.width), self.runtime.dtype)
+                ops.add_slabs(stream.x, pending, n, stream.pending_slabs, ctx.delta_slabs.stride(0), copy=rows)
+            elif pending is not None:
+                ops.add_slabs(stream.x, pending, n, stream.pending_slabs, ctx.delta_slabs.stride(0))
+            z = ctx.ws.alloc((ctx.max_slabs, n, self.cols), torch.float32)
+            parts = self.gate.slabs(ctx, rows, z)
+            g = ctx.ws.alloc((n, self.cols), self.runtime.dtype)
+            ops.token_gate(z[0], self.table, self.offset, self.dim, ctx.batch.token_ids[:n], g, self.runtime.status,
+                           n_partials=parts, partial_stride=z.stride(0))
+            stream.pending_slabs = self.proj.slabs(ctx, g, ctx.delta_slabs)
+        stream.pending, stream.pending_norm = ctx.delta, self.norm
 
 
 class DepthAveragedBlock(Part):
@@ -350,6 +475,8 @@ class HyperConnectionBlock(Part):
 
 
 register_part("block", "pre_norm", PreNormBlock)
+register_part("block", "parallel", ParallelBlock)
+register_part("block", "token_input", TokenInputBlock)
 register_part("block", "hyper_connections", HyperConnectionBlock)
 register_part("block", "sandwich_norm", SandwichNormBlock)
 register_part("block", "depth_averaged", DepthAveragedBlock)

@@ -17,13 +17,14 @@ class GatedMLP(FeedForward):
     there).  Gate and up weights are stacked at load, row by row alternately,
     so one product yields both and its epilogue can apply the activation to
     neighbouring outputs.  `activation` names one of the kernels' gate
-    activations (kernels.ops.ACTIVATIONS)."""
+    activations (kernels.ops.ACTIVATIONS); 'limited' takes its constants `limit` and `slope`
+    (kernels.ops.GateActivation)."""
     graph_safe = True
 
     DEFAULT_NAMES = ("gate_proj.weight", "up_proj.weight", "down_proj.weight")
 
     def __init__(self, runtime=None, prefix="", *, width: int, inner: int, activation: str = "silu",
-                 init_std: float = 0.02, names=DEFAULT_NAMES):
+                 init_std: float = 0.02, names=DEFAULT_NAMES, limit: float = 0.0, slope: float = 1.0):
         super().__init__(runtime, prefix)
         self.names = tuple(names)                # what the gate, up and down tensors are called behind the prefix
         if len(self.names) != 3:
@@ -31,7 +32,8 @@ class GatedMLP(FeedForward):
         if activation not in ops.ACTIVATIONS:
             raise ValueError(f"gated feed-forward: activation '{activation}' is not implemented "
                              f"({', '.join(sorted(ops.ACTIVATIONS))})")
-        self.activation = activation
+        self.activation = ops.GateActivation(activation, float(limit), float(slope))
+        ops.gate_arguments(self.activation)      # (constants that the activation cannot take are refused here)
         self.width, self.inner, self.init_std = int(width), int(inner), init_std
         self.gate_up = self.down = None
 

@@ -19,19 +19,24 @@ class RoutedExperts(FeedForward):
         the choice); the shares are the chosen scores themselves over their sum (+ 1e-20), times `weight_scale`;
       'sigmoid': scores s = sigmoid(z), every logit by itself; the `top` largest of s + br are chosen; the shares are
         the chosen scores as they are, times `weight_scale`.
+    `renormalize` (None: as the rule says): whether the two rules with scores divide the chosen ones by their sum.
+    `groups` / `keep_groups` (those two rules): the experts form `groups` equal groups of neighbours, a group counts as
+    its largest s + br, and only experts of the best `keep_groups` groups can be chosen (0: every expert).
     `share_on_input`: the share multiplies what the expert reads instead of what it gives, d = sum expert_e(share_e h)
     (the rows are scaled as they are laid side by side in expert order; with experts that are not linear in their
     input this is another function than the weighted sum of outputs).
     An expert is Wdown act(Wup h) with `activation` one of kernels.ops.PLAIN_ACTIVATIONS, or, with `gated`,
-    Wdown (act(Wgate h) * (Wup h)) with `activation` one of kernels.ops.ACTIVATIONS; experts have no biases.
+    Wdown (act(Wgate h) * (Wup h)) with `activation` one of kernels.ops.ACTIVATIONS ('limited' with its constants
+    `limit` and `slope`, kernels.ops.GateActivation); experts have no biases.
     `identity` (a count): that many more router outputs, behind the experts', stand for experts without weights
     whose output is their input h itself (times the share).
     A shared expert runs for every token and is added: with `shared_inner`, one of the experts' plain form times
-    sigmoid(w_sg . h), one number per token; with `shared` (a feed-forward PartSpec), that part's output as it is.
+    sigmoid(w_sg . h), one number per token; with `shared` (a feed-forward PartSpec), that part's output as it is, or,
+    with `shared_gate`, times such a sigmoid as well.
 
     Tensors behind the prefix: e<i>.up [inner, width], e<i>.down [width, inner] (gated: e<i>.gate as well), router
-    [experts + identity, width], `bias_name` [experts + identity] (if router_bias), and with `shared_inner`
-    shared.up, shared.down, shared.sg [1, width].
+    [experts + identity, width], `bias_name` [experts + identity] (if router_bias), with `shared_inner`
+    shared.up and shared.down, and with either kind of gate shared.sg [1, width].
 
     How a step runs: the router's logits (and the shared expert's gate) as one product, the choice (one warp a token),
     a counting sort of the (token, choice) pairs into expert order
@@ -45,7 +50,9 @@ class RoutedExperts(FeedForward):
                  activation: str = "relu_squared", shared_inner: int | None = None, router_bias: bool = True,
                  init_std: float = 0.02, router_std: float = 0.5, gated: bool = False,
                  rule: str = "softmax_of_chosen", weight_scale: float = 1.0, identity: int = 0,
-                 bias_name: str = "router.b", shared: PartSpec | None = None, share_on_input: bool = False):
+                 bias_name: str = "router.b", shared: PartSpec | None = None, share_on_input: bool = False,
+                 limit: float = 0.0, slope: float = 1.0, renormalize: bool | None = None, groups: int = 1,
+                 keep_groups: int = 0, shared_gate: bool = False):
         super().__init__(runtime, prefix)
         self.width, self.inner, self.E, self.K = int(width), int(inner), int(experts), int(top)
         self.identity = int(identity)
@@ -61,12 +68,27 @@ class RoutedExperts(FeedForward):
         if rule not in ops.ROUTER_RULES:
             raise ValueError(f"routed experts: rule '{rule}' is not one of {sorted(ops.ROUTER_RULES)}")
         self.activation, self.rule, self.weight_scale = activation, rule, float(weight_scale)
+        if self.gated:
+            self.activation = ops.GateActivation(activation, float(limit), float(slope))
+            ops.gate_arguments(self.activation)
+        self.renormalize, self.groups, self.keep_groups = renormalize, int(groups), int(keep_groups)
+        if self.groups < 1 or self.outputs % self.groups:
+            raise ValueError(f"routed experts: {self.outputs} experts do not form {self.groups} equal groups")
+        if self.keep_groups and rule == "softmax_of_chosen":
+            raise ValueError("routed experts: a choice within groups needs a rule that scores every expert")
+        if not 0 <= self.keep_groups <= self.groups or \
+                (self.keep_groups and self.K > self.keep_groups * (self.outputs // self.groups)):
+            raise ValueError(f"routed experts: top = {self.K} from {self.keep_groups} of {self.groups} groups of "
+                             f"{self.outputs // self.groups}")
         self.shared_inner = int(shared_inner) if shared_inner else 0
         if self.shared_inner and shared is not None:
             raise ValueError("routed experts: one shared expert, either of the experts' plain form or a part")
         if self.shared_inner and self.gated:
             raise ValueError("routed experts: beside gated experts the shared expert is a part of its own (`shared`)")
         self.shared = build_part(shared, runtime) if shared is not None else None
+        if shared_gate and shared is None:
+            raise ValueError("routed experts: a gate for a shared part that is not there")
+        self.token_gate = bool(self.shared_inner) or bool(shared_gate)    # sigmoid(w_sg . h) on the shared expert
         self.router_bias, self.init_std, self.router_std = bool(router_bias), init_std, router_std
         self.bias_name = bias_name
         self.up = self.down = self.router = self.router_b = None
@@ -89,6 +111,7 @@ class RoutedExperts(FeedForward):
         if self.shared_inner:
             specs[p + "shared.up"] = TensorSpec((self.shared_inner, self.width), init=init)
             specs[p + "shared.down"] = TensorSpec((self.width, self.shared_inner), init=init)
+        if self.token_gate:
             specs[p + "shared.sg"] = TensorSpec((1, self.width), init=init)
         return specs
 
@@ -103,7 +126,7 @@ class RoutedExperts(FeedForward):
         # the router and the shared expert's gate are one product: the gate's row lies behind the experts' rows
         # (then rows of zeros up to a multiple of 8, so that the product's float32 rows stay 16-byte aligned)
         rows = [tensors[p + "router"]]
-        if self.shared_inner:
+        if self.token_gate:
             rows.append(tensors[p + "shared.sg"].reshape(1, self.width).to(rows[0].dtype))
         have = sum(t.shape[0] for t in rows)
         if have % 8:
@@ -128,14 +151,16 @@ class RoutedExperts(FeedForward):
     def _shared_part(self, ctx, h, n):
         """The shared part's output: added to the stream by its own last product where that can be (None, 0, 0), else
         float32 shares in a buffer of its own (first share, how many, their stride)."""
-        kept = (ctx.delta_slabs, ctx.delta, ctx.pending_slabs)
+        kept = (ctx.delta_slabs, ctx.delta, ctx.pending_slabs, ctx.stream_x)
         sh = ctx.ws.alloc((ctx.max_slabs, n, self.width), torch.float32)
         ctx.delta_slabs, ctx.delta, ctx.pending_slabs = sh, sh[0], 1
+        if self.token_gate:
+            ctx.stream_x = None             # (what joins the stream is the gate times the output, not the output)
         try:
             self.shared.forward(ctx, h, sh[0])
             parts = ctx.pending_slabs
         finally:
-            ctx.delta_slabs, ctx.delta, ctx.pending_slabs = kept
+            ctx.delta_slabs, ctx.delta, ctx.pending_slabs, ctx.stream_x = kept
         return (None, 1, 0) if parts == 0 else (sh[0], parts, sh.stride(0))
 
     def forward(self, ctx, h, out):
@@ -151,12 +176,13 @@ class RoutedExperts(FeedForward):
         with ctx.ws.scope():
             chosen = ctx.ws.alloc((n, K), torch.int32)
             share = ctx.ws.alloc((n, K), torch.float32)
-            gate = ctx.ws.alloc((n,), torch.float32) if self.shared_inner else None
+            gate = ctx.ws.alloc((n,), torch.float32) if self.token_gate else None
             z = ctx.ws.alloc((ctx.max_slabs, n, self.router.out_features), torch.float32)
             parts = self.router.slabs(ctx, h[:n], z)
-            ops.moe_choose(z[0], self.router_b, self.outputs if self.shared_inner else -1, self.outputs, K, chosen,
+            ops.moe_choose(z[0], self.router_b, self.outputs if self.token_gate else -1, self.outputs, K, chosen,
                            share, gate, n_partials=parts, partial_stride=z.stride(0), rule=self.rule,
-                           weight_scale=self.weight_scale)
+                           weight_scale=self.weight_scale, renormalize=self.renormalize, groups=self.groups,
+                           keep_groups=self.keep_groups)
             place_token = ctx.ws.alloc((rows,), torch.int32)
             pair_place = ctx.ws.alloc((pairs,), torch.int32)
             tile_expert = ctx.ws.alloc((max_tiles,), torch.int32)

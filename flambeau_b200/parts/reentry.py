@@ -57,4 +57,40 @@ class ConcatLinearReentry(Part):
         stream.pending, stream.pending_slabs, stream.pending_norm = None, 0, None
 
 
+class AddReentry(Part):
+    """x <- x + x0 (the embedding output) + a learned vector of the pass, both float32: what a part left pending is
+    added first.  `first` says whether the first pass takes the embedding output in too (otherwise the passes behind it
+    do); with `step_name`, a tensor [passes, width] of that name holds the vectors, one for every pass."""
+    graph_safe = True
+    category = "reentry"
+
+    def __init__(self, runtime=None, prefix="", *, width: int, first: bool = False, step_name: str | None = None,
+                 passes: int = 0):
+        super().__init__(runtime, prefix)
+        self.width, self.first, self.step_name, self.passes = int(width), bool(first), step_name, int(passes)
+        if step_name is not None and self.passes < 1:
+            raise ValueError("a vector per pass needs the number of passes")
+        self.steps = None
+
+    def own_tensor_specs(self):
+        if self.step_name is None:
+            return {}
+        return {self.prefix + self.step_name: TensorSpec((self.passes, self.width), init=("normal", 0.1))}
+
+    def own_bind(self, tensors):
+        if self.step_name is not None:
+            self.steps = tensors[self.prefix + self.step_name].contiguous()
+
+    def forward(self, ctx, stream, x0, pass_index: int = 0) -> None:
+        n = ctx.n_tokens
+        if self.steps is not None and not 0 <= pass_index < self.passes:
+            raise ValueError(f"pass {pass_index} of a stretch that has vectors for {self.passes} passes")
+        stream.settle(ctx)
+        again = self.first or pass_index > 0
+        if again or self.steps is not None:
+            ops.add_row(stream.x[:n], self.steps[pass_index] if self.steps is not None else None,
+                        x0[:n] if again else None)
+
+
+register_part("reentry", "add", AddReentry)
 register_part("reentry", "concat_linear", ConcatLinearReentry)

@@ -31,8 +31,9 @@ class WeightError(ValueError):
 class FolderTensors:
     """The tensors of a model folder, checked against the model's wishes once and then fetched part by part."""
 
-    def __init__(self, folder, specs: dict, runtime):
-        """Raises WeightError listing everything that is off: missing, unexpected, wrong shape or kind."""
+    def __init__(self, folder, specs: dict, runtime, shared=()):
+        """Raises WeightError listing everything that is off: missing, unexpected, wrong shape or kind.  shared: names
+        that are fetched more than once and must stay one allocation."""
         self.files = ModelFiles(folder)
         self.specs, self.runtime = specs, runtime
         files = self.files
@@ -64,11 +65,13 @@ class FolderTensors:
         if missing or unexpected or wrong:
             files.close()
             raise WeightError(folder, sorted(missing), unexpected, wrong)
-        # a tensor that stands for several names (a tied head) is kept so that it stays one allocation
+        # a tensor that stands for several names (a tied head), or that several parts fetch, is kept so that it stays
+        # one allocation
         counts: dict = {}
         for src in self.source.values():
             counts[src] = counts.get(src, 0) + 1
         self._shared = {src: None for src, c in counts.items() if c > 1}
+        self._shared.update({self.source[name]: None for name in shared})
         self._warned = False
 
     def fetch(self, names) -> dict:
@@ -115,7 +118,7 @@ def load_model(folder, runtime):
     arch, cfg = load_config(folder)
     model = DecoderModel(arch.build_spec(cfg), runtime)
     model.config = cfg
-    ft = FolderTensors(folder, model.tensor_specs(), runtime)
+    ft = FolderTensors(folder, model.tensor_specs(), runtime, shared=model.shared_tensor_names())
     try:
         for part in model.parts():
             part.bind(ft.fetch(list(part.tensor_specs())))

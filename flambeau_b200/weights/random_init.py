@@ -90,6 +90,7 @@ def fill_random_on_device(model, seed: int = 0) -> None:
     all_specs = model.tensor_specs()
     shared: dict = {}                              # tensors that stand for another name too (a tied head)
     targets = {ts.alias_of for ts in all_specs.values() if ts.alias_of is not None and ts.alias_of in all_specs}
+    targets |= model.shared_tensor_names()         # and those that several parts read
     for part in model.parts():
         tensors = {}
         for name, ts in part.tensor_specs().items():
