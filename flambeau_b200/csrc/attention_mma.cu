@@ -279,13 +279,21 @@ attention_mma_kernel(const __grid_constant__ AttnArgs a) {
         }
         // ---- scale, mask, online softmax ----
         const float to_log2 = a.cap_log2e > 0.0f ? 1.0f : a.scale_log2e;
-        if (a.cap_log2e > 0.0f) {
+        if (a.cap_log2e > FB_SOFTCAP_DIRECT) {
 #pragma unroll
             for (int rb = 0; rb < R; ++rb)
 #pragma unroll
                 for (int nb = 0; nb < NSB; ++nb)
 #pragma unroll
                     for (int e = 0; e < 4; ++e) s[rb][nb][e] = fb_softcap(s[rb][nb][e] * a.scale_over_cap, a.cap_log2e);
+        } else if (a.cap_log2e > 0.0f) {
+            const float to_x = a.scale_over_cap * 2.8853900817779268f;
+#pragma unroll
+            for (int rb = 0; rb < R; ++rb)
+#pragma unroll
+                for (int nb = 0; nb < NSB; ++nb)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) s[rb][nb][e] = fb_softcap_direct(s[rb][nb][e] * to_x, a.cap_log2e);
         }
         uint32_t pa[R][KT / 16][4];            // the probabilities as A fragments of P V
 #pragma unroll

@@ -178,6 +178,17 @@ __device__ __forceinline__ float fb_softcap(float y, float cap) {
     return copysignf(cap * (a < 0.2f ? small : big), y);
 }
 
+// The same where the cap is at most FB_SOFTCAP_DIRECT (in base-2 units): cap (1 - 2 / (1 + 2^x)) with x = 2 log2(e) score /
+// cap.  Its absolute error is about 2e-7 of the cap, which for caps of tens is far below what scores of 16-bit queries and
+// keys carry; five instructions.
+constexpr float FB_SOFTCAP_DIRECT = 400.0f;
+__device__ __forceinline__ float fb_softcap_direct(float x, float cap) {
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));       // (e = inf: 0; e = 0: 1)
+    return fmaf(-2.0f * cap, r, cap);
+}
+
 // ---- reductions -------------------------------------------------------------
 __device__ __forceinline__ float fb_warp_sum(float v) {
 #pragma unroll

@@ -17,12 +17,14 @@
 //                padded order its token (-1: padding), for every pair its place, for every row tile its expert
 //                (-1: unused).  Sizes are upper bounds known on the host, so nothing has to come back from the device
 //   moe_combine  per token: sum_k weight_k * expert_out[place of (token, k)] + gate * shared_out; a chosen expert
-//                beyond the ones that have weights (an identity expert) hands the token's own input on
+//                beyond the ones that have weights (an identity expert) hands the token's own input on.  The sum
+//                replaces what the output row holds, or is added to it (`accumulate`: the row is the residual stream's)
 #include "common.cuh"
 
 constexpr int MOE_MAX_LOGITS_PER_LANE = 16;            // 512 experts at most
 
-template <typename TW>
+// R: logits a lane holds (E <= 32 R)
+template <typename TW, int R>
 __global__ void __launch_bounds__(128)
 moe_choose_kernel(const float* __restrict__ z_in, long z_stride, int n_partials, long partial_stride,
                   const TW* __restrict__ br, int gate_col, int n, int E, int K, int* __restrict__ chosen,
@@ -35,13 +37,13 @@ moe_choose_kernel(const float* __restrict__ z_in, long z_stride, int n_partials,
     if (row >= n) return;
     const float* zr = z_in + (size_t)row * z_stride;
     auto logit = [&](int c) { return fb_slab_sum(zr, c, n_partials, partial_stride); };
-    float z[MOE_MAX_LOGITS_PER_LANE];                  // lane l keeps the logits of experts l, l + 32, ...
+    float z[R];                  // lane l keeps the logits of experts l, l + 32, ...
     if (rule == 1 || rule == 2) {
         // scores over all experts first; the bias only moves the choice
-        float s[MOE_MAX_LOGITS_PER_LANE];
+        float s[R];
         float top = -INFINITY;
 #pragma unroll
-        for (int r = 0; r < MOE_MAX_LOGITS_PER_LANE; ++r) {
+        for (int r = 0; r < R; ++r) {
             const int e = lane + 32 * r;
             s[r] = e < E ? logit(e) : -INFINITY;
             top = fmaxf(top, s[r]);
@@ -50,20 +52,20 @@ moe_choose_kernel(const float* __restrict__ z_in, long z_stride, int n_partials,
             top = fb_warp_max(top);
             float sum = 0.0f;
 #pragma unroll
-            for (int r = 0; r < MOE_MAX_LOGITS_PER_LANE; ++r) {
+            for (int r = 0; r < R; ++r) {
                 s[r] = lane + 32 * r < E ? expf(s[r] - top) : 0.0f;
                 sum += s[r];
             }
             sum = fb_warp_sum(sum);
 #pragma unroll
-            for (int r = 0; r < MOE_MAX_LOGITS_PER_LANE; ++r) s[r] = s[r] / sum;
+            for (int r = 0; r < R; ++r) s[r] = s[r] / sum;
         } else {
 #pragma unroll
-            for (int r = 0; r < MOE_MAX_LOGITS_PER_LANE; ++r)
+            for (int r = 0; r < R; ++r)
                 s[r] = lane + 32 * r < E ? 1.0f / (1.0f + expf(-s[r])) : 0.0f;
         }
 #pragma unroll
-        for (int r = 0; r < MOE_MAX_LOGITS_PER_LANE; ++r) {
+        for (int r = 0; r < R; ++r) {
             const int e = lane + 32 * r;
             z[r] = e < E ? s[r] + (br ? fb_to_float(br[e]) : 0.0f) : -INFINITY;
         }
@@ -75,7 +77,7 @@ moe_choose_kernel(const float* __restrict__ z_in, long z_stride, int n_partials,
                 float best = -INFINITY;
                 int best_e = 0x7fffffff;
 #pragma unroll
-                for (int r = 0; r < MOE_MAX_LOGITS_PER_LANE; ++r)
+                for (int r = 0; r < R; ++r)
                     if (!(in >> r & 1u) && z[r] > best) { best = z[r]; best_e = lane + 32 * r; }
 #pragma unroll
                 for (int off = 16; off > 0; off >>= 1) {
@@ -85,11 +87,11 @@ moe_choose_kernel(const float* __restrict__ z_in, long z_stride, int n_partials,
                 }
                 const int group = best_e / group_size;
 #pragma unroll
-                for (int r = 0; r < MOE_MAX_LOGITS_PER_LANE; ++r)
+                for (int r = 0; r < R; ++r)
                     if ((lane + 32 * r) / group_size == group) in |= 1u << r;
             }
 #pragma unroll
-            for (int r = 0; r < MOE_MAX_LOGITS_PER_LANE; ++r)
+            for (int r = 0; r < R; ++r)
                 if (!(in >> r & 1u)) z[r] = -INFINITY;
         }
         float total = 0.0f, mine = 0.0f;               // lane k keeps the k-th chosen score
@@ -97,7 +99,7 @@ moe_choose_kernel(const float* __restrict__ z_in, long z_stride, int n_partials,
             float best = -INFINITY, best_s = 0.0f;
             int best_e = 0x7fffffff;
 #pragma unroll
-            for (int r = 0; r < MOE_MAX_LOGITS_PER_LANE; ++r) {
+            for (int r = 0; r < R; ++r) {
                 const int e = lane + 32 * r;
                 if (e < E && (z[r] > best)) { best = z[r]; best_e = e; best_s = s[r]; }
             }
@@ -109,7 +111,7 @@ moe_choose_kernel(const float* __restrict__ z_in, long z_stride, int n_partials,
                 if (ob > best || (ob == best && oe < best_e)) { best = ob; best_e = oe; best_s = os; }
             }
 #pragma unroll
-            for (int r = 0; r < MOE_MAX_LOGITS_PER_LANE; ++r)
+            for (int r = 0; r < R; ++r)
                 if (best_e == lane + 32 * r) z[r] = -INFINITY;           // taken
             total += best_s;
             if (lane == k) mine = best_s;
@@ -120,7 +122,7 @@ moe_choose_kernel(const float* __restrict__ z_in, long z_stride, int n_partials,
         return;
     }
 #pragma unroll
-    for (int r = 0; r < MOE_MAX_LOGITS_PER_LANE; ++r) {
+    for (int r = 0; r < R; ++r) {
         const int e = lane + 32 * r;
         z[r] = e < E ? logit(e) + (br ? fb_to_float(br[e]) : 0.0f) : -INFINITY;
     }
@@ -130,7 +132,7 @@ moe_choose_kernel(const float* __restrict__ z_in, long z_stride, int n_partials,
         float best = -INFINITY;
         int best_e = 0x7fffffff;
 #pragma unroll
-        for (int r = 0; r < MOE_MAX_LOGITS_PER_LANE; ++r) {
+        for (int r = 0; r < R; ++r) {
             const int e = lane + 32 * r;
             if (e < E && (z[r] > best)) { best = z[r]; best_e = e; }     // ascending e: the lower index stays on a tie
         }
@@ -141,7 +143,7 @@ moe_choose_kernel(const float* __restrict__ z_in, long z_stride, int n_partials,
             if (ob > best || (ob == best && oe < best_e)) { best = ob; best_e = oe; }
         }
 #pragma unroll
-        for (int r = 0; r < MOE_MAX_LOGITS_PER_LANE; ++r)
+        for (int r = 0; r < R; ++r)
             if (best_e == lane + 32 * r) z[r] = -INFINITY;               // taken
         if (k == 0) first = best;
         const float p = expf(best - first);            // the first chosen logit is the largest
@@ -196,7 +198,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ expert_out, long ex
                                    const int* __restrict__ pair_place, const float* __restrict__ share, int K,
                                    const float* __restrict__ shared_out, int shared_partials, long shared_partial_stride,
                                    const float* __restrict__ gate, float* __restrict__ out, int n, int D,
-                                   const T* __restrict__ pass_on, long pass_stride) {
+                                   const T* __restrict__ pass_on, long pass_stride, int accumulate) {
     fb_pdl_launch_dependents();
     fb_pdl_wait();
     const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -214,7 +216,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ expert_out, long ex
         for (int p = 0; p < shared_partials; ++p) s += shared_out[(size_t)p * shared_partial_stride + idx];
         acc = fmaf(gate ? gate[row] : 1.0f, s, acc);
     }
-    out[idx] = acc;
+    out[idx] = accumulate ? out[idx] + acc : acc;
 }
 
 // out[place] = h[place_token[place]] (a row of zeros where the place is padding): the tokens side by side in expert
@@ -301,9 +303,16 @@ FB_API int fb_moe_choose(const float* z, long long z_stride, int n_partials, lon
     FB_REQUIRE(z_stride >= E && z_stride > gate_col, "router: logit rows are too short");
     if (n == 0) return 0;
     if (n_partials < 1) n_partials = 1;
-    FB_DISPATCH_DTYPE(w_dtype, TW,
-        (fb_launch((moe_choose_kernel<TW>), dim3((n + 3) / 4), dim3(128), 0, stream, z, (long)z_stride, n_partials,
-                   (long)partial_stride, (const TW*)br, gate_col, n, E, K, chosen, share, gate, rule, weight_scale, renorm, E / n_groups, keep_groups)));
+#define FB_CHOOSE(R_)                                                                                                 \
+    FB_DISPATCH_DTYPE(w_dtype, TW,                                                                                    \
+        (fb_launch((moe_choose_kernel<TW, R_>), dim3((n + 3) / 4), dim3(128), 0, stream, z, (long)z_stride, n_partials, \
+                   (long)partial_stride, (const TW*)br, gate_col, n, E, K, chosen, share, gate, rule, weight_scale,   \
+                   renorm, E / n_groups, keep_groups)))
+    if (E <= 32) FB_CHOOSE(1);
+    else if (E <= 64) FB_CHOOSE(2);
+    else if (E <= 128) FB_CHOOSE(4);
+    else FB_CHOOSE(MOE_MAX_LOGITS_PER_LANE);
+#undef FB_CHOOSE
     return fb_check_launch("moe_choose");
 }
 
@@ -331,7 +340,7 @@ __global__ void moe_combine_vec_kernel(const float* __restrict__ expert_out, lon
                                        const float* __restrict__ shared_out, int shared_partials,
                                        long shared_partial_stride, const float* __restrict__ gate,
                                        float* __restrict__ out, int n, int D, const T* __restrict__ pass_on,
-                                       long pass_stride) {
+                                       long pass_stride, int accumulate) {
     fb_pdl_launch_dependents();
     fb_pdl_wait();
     const int nvec = D >> 2;
@@ -339,6 +348,8 @@ __global__ void moe_combine_vec_kernel(const float* __restrict__ expert_out, lon
     if (idx >= (size_t)n * nvec) return;
     const int row = (int)(idx / nvec), c = (int)(idx - (size_t)row * nvec) * 4;
     float4 acc = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    float4 held = acc;
+    if (accumulate) held = *reinterpret_cast<const float4*>(out + (size_t)row * D + c);
     for (int k = 0; k < K; ++k) {
         const int at = pair_place[(size_t)row * K + k];
         if (at < 0 && !pass_on) continue;
@@ -362,16 +373,17 @@ __global__ void moe_combine_vec_kernel(const float* __restrict__ expert_out, lon
         const float gt = gate ? gate[row] : 1.0f;
         acc.x = fmaf(gt, s.x, acc.x); acc.y = fmaf(gt, s.y, acc.y); acc.z = fmaf(gt, s.z, acc.z); acc.w = fmaf(gt, s.w, acc.w);
     }
+    acc.x += held.x; acc.y += held.y; acc.z += held.z; acc.w += held.w;
     *reinterpret_cast<float4*>(out + (size_t)row * D + c) = acc;
 }
 
 // pass_on (optional, [n, D] rows `pass_stride` apart, dtype code `pass_dtype`): what a pair without a place (a chosen
 // expert that has no weights) contributes, times its share.  share = nullptr: every pair counts once (the shares
-// have scaled the experts' inputs already).
+// have scaled the experts' inputs already).  accumulate: the sum is added to what `out` holds.
 FB_API int fb_moe_combine(const float* expert_out, long long expert_stride, const int* pair_place, const float* share,
                           int K, const float* shared_out, int shared_partials, long long shared_partial_stride,
                           const float* gate, float* out, int n, int D, const void* pass_on, int pass_dtype,
-                          long long pass_stride, cudaStream_t stream) {
+                          long long pass_stride, int accumulate, cudaStream_t stream) {
     FB_REQUIRE(n >= 0 && D > 0 && K > 0, "moe_combine: bad sizes");
     if (n == 0) return 0;
     if (!pass_on) pass_dtype = FB_F32;
@@ -382,13 +394,13 @@ FB_API int fb_moe_combine(const float* expert_out, long long expert_stride, cons
             (fb_launch((moe_combine_vec_kernel<T>), dim3((unsigned)((total4 + 255) / 256)), dim3(256), 0, stream,
                        expert_out, (long)expert_stride, pair_place, share, K, shared_out,
                        shared_partials < 1 ? 1 : shared_partials, (long)shared_partial_stride, gate, out, n, D,
-                       (const T*)pass_on, (long)pass_stride)));
+                       (const T*)pass_on, (long)pass_stride, accumulate)));
         return fb_check_launch("moe_combine");
     }
     const size_t total = (size_t)n * D;
     FB_DISPATCH_DTYPE(pass_dtype, T,
         (fb_launch((moe_combine_kernel<T>), dim3((unsigned)((total + 255) / 256)), dim3(256), 0, stream, expert_out,
                    (long)expert_stride, pair_place, share, K, shared_out, shared_partials < 1 ? 1 : shared_partials,
-                   (long)shared_partial_stride, gate, out, n, D, (const T*)pass_on, (long)pass_stride)));
+                   (long)shared_partial_stride, gate, out, n, D, (const T*)pass_on, (long)pass_stride, accumulate)));
     return fb_check_launch("moe_combine");
 }

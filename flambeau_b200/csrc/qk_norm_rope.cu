@@ -117,10 +117,13 @@ qk_norm_rope_kv_write_kernel(const float* __restrict__ proj, long proj_stride, i
     }
 }
 
-// One warp per (row, head): heads 0 .. nh - 1 are queries, the nkv behind them keys, the nkv behind those values (none
-// where the values are the keys as projected: the key's warp then writes both).  NV = float4 a lane holds of a head.
+// A warp takes HPW neighbouring heads of a row: heads 0 .. nh - 1 are queries, the nkv behind them keys, the nkv behind
+// those values (none where the values are the keys as projected: the key's warp then writes both).  NV = float4 a lane
+// holds of a head.  Every load of the warp's heads is issued before the first use.  The two members of a rotated pair lie
+// 2 * half / 8 lanes apart where NV is 1 and half a multiple of 4 (one exchange between lanes); otherwise they meet in the
+// warp's stretch of shared memory.
 constexpr int QKR_WARPS = 8;
-template <typename TW, typename T, int NV>
+template <typename TW, typename T, int NV, int HPW>
 __global__ void __launch_bounds__(32 * QKR_WARPS)
 qk_norm_rope_heads_kernel(const float* __restrict__ proj, long proj_stride, int n_partials, long partial_stride,
                           const TW* __restrict__ q_weight, const TW* __restrict__ k_weight, float eps,
@@ -131,89 +134,153 @@ qk_norm_rope_heads_kernel(const float* __restrict__ proj, long proj_stride, int 
                           T* __restrict__ v_pool, int page_size, int n_pages, int n, int nh, int nkv, int hd, int vd,
                           int v_off, int v_is_k, int write_kv, int* status) {
     fb_pdl_launch_dependents();
-    fb_pdl_wait();
-    extern __shared__ float sh[];                      // [QKR_WARPS][hd]
+    extern __shared__ float sh[];                      // [QKR_WARPS][hd], where pairs meet in shared memory
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int per_row = nh + (write_kv ? (v_is_k ? nkv : 2 * nkv) : 0);
+    const int groups = (per_row + HPW - 1) / HPW;
     const long item = (long)blockIdx.x * QKR_WARPS + warp;
-    if (item >= (long)n * per_row) return;
-    const int row = (int)(item / per_row), h = (int)(item - (long)row * per_row);
-    const bool is_q = h < nh, is_v = h >= nh + nkv;
-    const int g = is_q ? h : is_v ? h - nh - nkv : h - nh;
-    const int width = is_v ? vd : hd, nvec = width >> 2;
-    const float* src = proj + (size_t)row * proj_stride + (is_q ? (size_t)h * hd : is_v ? (size_t)v_off + (size_t)g * vd
-                                                                                        : (size_t)(nh + g) * hd);
-    float4 x[NV];
+    const int row = (int)(item / groups), h0 = (int)(item - (long)row * groups) * HPW;
+    const bool by_lanes = NV == 1 && (half & 3) == 0;
+    float4 wq[NV], wk[NV];                             // the norms' weights (parameters, not of this step)
+    if (q_weight) {
 #pragma unroll
-    for (int i = 0; i < NV; ++i) {
-        const int c = lane + 32 * i;
-        x[i] = c < nvec ? slab_sum4(src + 4 * c, n_partials, partial_stride) : make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int i = 0; i < NV; ++i) {
+            const int c = lane + 32 * i;
+            wq[i] = wk[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (c >= hd >> 2) continue;
+            wq[i] = Vec4<TW>::load(q_weight + 4 * c);
+            wk[i] = Vec4<TW>::load(k_weight + 4 * c);
+            wq[i].x += weight_offset; wq[i].y += weight_offset; wq[i].z += weight_offset; wq[i].w += weight_offset;
+            wk[i].x += weight_offset; wk[i].y += weight_offset; wk[i].z += weight_offset; wk[i].w += weight_offset;
+        }
     }
-    T* k_dst = nullptr;
-    T* v_dst = nullptr;
-    if (!is_q) {
+    fb_pdl_wait();
+    if (row >= n) return;
+    float4 x[HPW][NV];
+#pragma unroll
+    for (int j = 0; j < HPW; ++j) {
+        const int h = h0 + j;
+        const bool is_v = h >= nh + nkv;
+        const int nvec = (is_v ? vd : hd) >> 2;
+        const float* src = proj + (size_t)row * proj_stride +
+                           (is_v ? (size_t)v_off + (size_t)(h - nh - nkv) * vd : (size_t)h * hd);
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int c = lane + 32 * i;
+            x[j][i] = h < per_row && c < nvec ? Vec4<float>::load(src + 4 * c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+    }
+    // the pairs' cosines and sines: this lane's four columns are four pairs, first members for columns below `half`
+    float4 cs = make_float4(0.f, 0.f, 0.f, 0.f), sn = cs;
+    const bool turns = by_lanes && 4 * lane < 2 * half, second = 4 * lane >= half;
+    if (turns) {
+        const size_t at = (size_t)row * half + 4 * lane - (second ? half : 0);
+        cs = Vec4<float>::load(cos_t + at);
+        sn = Vec4<float>::load(sin_t + at);
+        if (!second) { sn.x = -sn.x; sn.y = -sn.y; sn.z = -sn.z; sn.w = -sn.w; }
+    }
+    size_t cache_row = 0;                              // + head * page_size: the token's row in a pool
+    bool cached = false;
+    if (h0 + HPW > nh && write_kv) {
         const int p = positions[row], seq = row_seq[row];
         const int entry = fb_table_column(p / page_size, table_base ? table_base[seq] : 0, table_head);
         const int page = (entry >= 0 && entry < table_stride) ? block_table[(size_t)seq * table_stride + entry] : -1;
-        if (page < 0 || page >= n_pages) {
-            if (lane == 0) atomicOr(status, FB_STATUS_BAD_PAGE);
-            return;
-        }
-        const size_t at = ((size_t)page * nkv + g) * page_size + (p % page_size);
-        k_dst = k_pool + at * hd;
-        v_dst = v_pool + at * vd;
+        cached = page >= 0 && page < n_pages;
+        if (!cached && lane == 0) atomicOr(status, FB_STATUS_BAD_PAGE);
+        cache_row = (size_t)page * nkv * page_size + (p % page_size);
     }
-    if (is_v || (!is_q && v_is_k)) {
+    if (n_partials > 1) {
+        // one head: its shares eight at a time; several: share after share, a load of every head in flight
+        for (int p0 = 1; p0 < n_partials; p0 += HPW == 1 ? n_partials - 1 : 1) {
 #pragma unroll
-        for (int i = 0; i < NV; ++i) {
-            const int c = lane + 32 * i;
-            if (c < nvec) Vec4<T>::store(v_dst + 4 * c, x[i]);
-        }
-        if (is_v) return;
-    }
-    const TW* w = is_q ? q_weight : k_weight;
-    if (w) {
-        float s = 0.0f;
+            for (int j = 0; j < HPW; ++j) {
+                const int h = h0 + j;
+                const bool is_v = h >= nh + nkv;
+                const int nvec = (is_v ? vd : hd) >> 2;
+                const float* src = proj + (size_t)row * proj_stride + (size_t)p0 * partial_stride +
+                                   (is_v ? (size_t)v_off + (size_t)(h - nh - nkv) * vd : (size_t)h * hd);
 #pragma unroll
-        for (int i = 0; i < NV; ++i) s += x[i].x * x[i].x + x[i].y * x[i].y + x[i].z * x[i].z + x[i].w * x[i].w;
-        const float f = 1.0f / sqrtf(fb_warp_sum(s) / (float)hd + eps);
-#pragma unroll
-        for (int i = 0; i < NV; ++i) {
-            const int c = lane + 32 * i;
-            if (c >= nvec) continue;
-            const float4 wv = Vec4<TW>::load(w + 4 * c);
-            x[i].x *= f * (wv.x + weight_offset); x[i].y *= f * (wv.y + weight_offset);
-            x[i].z *= f * (wv.z + weight_offset); x[i].w *= f * (wv.w + weight_offset);
-        }
-    }
-    if (half > 0) {
-        float* mine = sh + (size_t)warp * hd;
-#pragma unroll
-        for (int i = 0; i < NV; ++i) {
-            const int c = lane + 32 * i;
-            if (4 * c < 2 * half) Vec4<float>::store(mine + 4 * c, x[i]);
-        }
-        __syncwarp();
-        const float* cs = cos_t + (size_t)row * half;
-        const float* sn = sin_t + (size_t)row * half;
-#pragma unroll
-        for (int i = 0; i < NV; ++i) {
-            const int d0 = 4 * (lane + 32 * i);
-            if (d0 >= 2 * half) continue;
-            float* xe = reinterpret_cast<float*>(&x[i]);
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int d = d0 + e;
-                if (d < half) xe[e] = xe[e] * cs[d] - mine[d + half] * sn[d];
-                else if (d < 2 * half) xe[e] = xe[e] * cs[d - half] + mine[d - half] * sn[d - half];
+                for (int i = 0; i < NV; ++i) {
+                    const int c = lane + 32 * i;
+                    if (h >= per_row || c >= nvec) continue;
+                    const float4 more = HPW == 1 ? slab_sum4(src + 4 * c, n_partials - 1, partial_stride)
+                                                 : Vec4<float>::load(src + 4 * c);
+                    x[j][i].x += more.x; x[j][i].y += more.y; x[j][i].z += more.z; x[j][i].w += more.w;
+                }
             }
         }
     }
-    T* dst = is_q ? q_out + (size_t)row * q_out_stride + (size_t)h * hd : k_dst;
 #pragma unroll
-    for (int i = 0; i < NV; ++i) {
-        const int c = lane + 32 * i;
-        if (c < nvec) Vec4<T>::store(dst + 4 * c, x[i]);
+    for (int j = 0; j < HPW; ++j) {
+        const int h = h0 + j;
+        if (h >= per_row) break;
+        const bool is_q = h < nh, is_v = h >= nh + nkv;
+        const int g = is_q ? h : is_v ? h - nh - nkv : h - nh;
+        const int nvec = (is_v ? vd : hd) >> 2;
+        if (!is_q && !cached) continue;
+        const size_t at = is_q ? 0 : cache_row + (size_t)g * page_size;
+        if (is_v || (!is_q && v_is_k)) {
+            T* v_dst = v_pool + at * vd;
+#pragma unroll
+            for (int i = 0; i < NV; ++i) {
+                const int c = lane + 32 * i;
+                if (c < nvec) Vec4<T>::store(v_dst + 4 * c, x[j][i]);
+            }
+            if (is_v) continue;
+        }
+        if (q_weight) {
+            float s = 0.0f;
+#pragma unroll
+            for (int i = 0; i < NV; ++i)
+                s += x[j][i].x * x[j][i].x + x[j][i].y * x[j][i].y + x[j][i].z * x[j][i].z + x[j][i].w * x[j][i].w;
+            const float f = 1.0f / sqrtf(fb_warp_sum(s) / (float)hd + eps);
+#pragma unroll
+            for (int i = 0; i < NV; ++i) {
+                const float4 w = is_q ? wq[i] : wk[i];
+                x[j][i].x *= f * w.x; x[j][i].y *= f * w.y; x[j][i].z *= f * w.z; x[j][i].w *= f * w.w;
+            }
+        }
+        if (by_lanes) {
+            if (half > 0) {
+                const int mate = (second ? lane - (half >> 2) : lane + (half >> 2)) & 31;
+                float4 o;
+                o.x = __shfl_sync(0xffffffffu, x[j][0].x, mate); o.y = __shfl_sync(0xffffffffu, x[j][0].y, mate);
+                o.z = __shfl_sync(0xffffffffu, x[j][0].z, mate); o.w = __shfl_sync(0xffffffffu, x[j][0].w, mate);
+                if (turns) {
+                    x[j][0].x = x[j][0].x * cs.x + o.x * sn.x; x[j][0].y = x[j][0].y * cs.y + o.y * sn.y;
+                    x[j][0].z = x[j][0].z * cs.z + o.z * sn.z; x[j][0].w = x[j][0].w * cs.w + o.w * sn.w;
+                }
+            }
+        } else if (half > 0) {
+            float* mine = sh + (size_t)warp * hd;
+            __syncwarp();                              // (the head before has been read)
+#pragma unroll
+            for (int i = 0; i < NV; ++i) {
+                const int c = lane + 32 * i;
+                if (c < nvec && 4 * c < 2 * half) Vec4<float>::store(mine + 4 * c, x[j][i]);
+            }
+            __syncwarp();
+            const float* ct = cos_t + (size_t)row * half;
+            const float* st = sin_t + (size_t)row * half;
+#pragma unroll
+            for (int i = 0; i < NV; ++i) {
+                const int d0 = 4 * (lane + 32 * i);
+                if (d0 >= 2 * half) continue;
+                float* xe = reinterpret_cast<float*>(&x[j][i]);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int d = d0 + e;
+                    if (d < half) xe[e] = xe[e] * ct[d] - mine[d + half] * st[d];
+                    else if (d < 2 * half) xe[e] = xe[e] * ct[d - half] + mine[d - half] * st[d - half];
+                }
+            }
+        }
+        T* dst = is_q ? q_out + (size_t)row * q_out_stride + (size_t)h * hd : k_pool + at * hd;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int c = lane + 32 * i;
+            if (c < nvec) Vec4<T>::store(dst + 4 * c, x[j][i]);
+        }
     }
 }
 
@@ -247,20 +314,23 @@ FB_API int fb_qk_norm_rope_kv_write(const float* proj, long long proj_stride, in
         aligned(q_weight, 4 * wsize) && aligned(k_weight, 4 * wsize)) {
         if (scope == FB_QK_NORM_NONE) q_weight = k_weight = nullptr;
         const int v_is_k = v_off == k_off ? 1 : 0;
-        const long items = (long)n * (nh + (write_kv ? (v_is_k ? nkv : 2 * nkv) : 0));
+        // (a few rows: one head a warp, so that the heads spread over the device; a portion: four, for loads in flight)
+        const int hpw = n <= 64 ? 1 : 4;
+        const int per_row = nh + (write_kv ? (v_is_k ? nkv : 2 * nkv) : 0);
+        const long items = (long)n * ((per_row + hpw - 1) / hpw);
         const unsigned blocks = (unsigned)((items + QKR_WARPS - 1) / QKR_WARPS);
         const size_t smem_h = (size_t)QKR_WARPS * hd * sizeof(float);
         const int widest = hd > vd ? hd : vd;
-#define FB_QKR_HEADS(NV_)                                                                                             \
+#define FB_QKR_HEADS(NV_, HPW_)                                                                                       \
         FB_DISPATCH_DTYPE(w_dtype, TW, FB_DISPATCH_DTYPE(out_dtype, T,                                                \
-            (fb_launch((qk_norm_rope_heads_kernel<TW, T, NV_>), dim3(blocks), dim3(32 * QKR_WARPS), smem_h, stream, proj, \
-                       (long)proj_stride, n_partials, (long)partial_stride, (const TW*)q_weight, (const TW*)k_weight, eps, \
-                       weight_offset, cos_t, sin_t, half, (T*)q_out, (long)q_out_stride, positions, row_seq, block_table, \
+            (fb_launch((qk_norm_rope_heads_kernel<TW, T, NV_, HPW_>), dim3(blocks), dim3(32 * QKR_WARPS), smem_h, stream, \
+                       proj, (long)proj_stride, n_partials, (long)partial_stride, (const TW*)q_weight, (const TW*)k_weight, \
+                       eps, weight_offset, cos_t, sin_t, half, (T*)q_out, (long)q_out_stride, positions, row_seq, block_table, \
                        table_stride, table_base, table_head, (T*)k_pool, (T*)v_pool, page_size, n_pages, n, nh, nkv, hd, vd, \
                        v_off, v_is_k, write_kv, status))))
-        if (widest <= 128) FB_QKR_HEADS(1);
-        else if (widest <= 256) FB_QKR_HEADS(2);
-        else FB_QKR_HEADS(4);
+        if (widest <= 128) { if (hpw == 1) FB_QKR_HEADS(1, 1); else FB_QKR_HEADS(1, 4); }
+        else if (widest <= 256) { if (hpw == 1) FB_QKR_HEADS(2, 1); else FB_QKR_HEADS(2, 4); }
+        else { if (hpw == 1) FB_QKR_HEADS(4, 1); else FB_QKR_HEADS(4, 4); }
 #undef FB_QKR_HEADS
         return fb_check_launch("qk_norm_rope_kv_write");
     }

@@ -80,27 +80,37 @@ FB_API int fb_embedding_pairs(const void* table, const void* pairs, int table_dt
     return fb_check_launch("embedding_pairs");
 }
 
-template <typename TT, typename TO>
+template <typename TT, typename TO, int VEC>
 __global__ void __launch_bounds__(256)
 token_gate_kernel(const float* __restrict__ z, long z_stride, int n_partials, long partial_stride,
                   const TT* __restrict__ table, long table_stride, int offset, const int* __restrict__ ids, int V,
                   TO* __restrict__ out, int n, int dim, int cols, int* status) {
     fb_pdl_launch_dependents();
-    fb_pdl_wait();
+    const int per = cols / VEC;
     const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (idx >= (size_t)n * cols) return;
-    const int t = (int)(idx / cols), c = (int)(idx - (size_t)t * cols);
-    float g = 0.0f;
-    if (c < dim) {
-        int id = ids[t];
-        if (id < 0 || id >= V) {
-            atomicOr(status, FB_STATUS_BAD_TOKEN);
-            id = 0;
-        }
-        const float e = fb_to_float(table[(size_t)id * table_stride + offset + c]);
-        g = fb_gelu_tanh(fb_slab_sum(z + (size_t)t * z_stride, c, n_partials, partial_stride)) * e;
+    const int t = (int)(idx / per), c = (int)(idx - (size_t)t * per) * VEC;
+    fb_pdl_wait();
+    if (t >= n) return;
+    int id = ids[t];
+    if (id < 0 || id >= V) {
+        atomicOr(status, FB_STATUS_BAD_TOKEN);
+        id = 0;
     }
-    out[idx] = fb_from_float<TO>(g);
+    const TT* e = table + (size_t)id * table_stride + offset + c;
+    const float* zr = z + (size_t)t * z_stride + c;
+    TO* o = out + (size_t)t * cols + c;
+    if constexpr (VEC == 4) {                          // dim is a multiple of 4: a thread's columns are all in or all out
+        float4 g = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c < dim) {
+            const float4 u = Vec4<TT>::load(e);
+            g = slab_sum4(zr, n_partials, partial_stride);
+            g.x = fb_gelu_tanh(g.x) * u.x; g.y = fb_gelu_tanh(g.y) * u.y;
+            g.z = fb_gelu_tanh(g.z) * u.z; g.w = fb_gelu_tanh(g.w) * u.w;
+        }
+        Vec4<TO>::store(o, g);
+    } else {
+        o[0] = fb_from_float<TO>(c < dim ? fb_gelu_tanh(fb_slab_sum(zr, 0, n_partials, partial_stride)) * fb_to_float(e[0]) : 0.0f);
+    }
 }
 
 // z: float32 [n, >= dim] (possibly shares); table [V, table_stride], of which a layer reads `dim` columns from `offset`
@@ -112,10 +122,18 @@ FB_API int fb_token_gate(const float* z, long long z_stride, int n_partials, lon
     FB_REQUIRE(offset >= 0 && table_stride >= (long long)offset + dim, "token_gate: the table's rows are too short");
     if (n == 0) return 0;
     if (n_partials < 1) n_partials = 1;
-    const size_t total = (size_t)n * cols;
-    FB_DISPATCH_DTYPE(table_dtype, TT, FB_DISPATCH_DTYPE(out_dtype, TO,
-        (fb_launch((token_gate_kernel<TT, TO>), (unsigned)((total + 255) / 256), 256, 0, stream, z, (long)z_stride,
-                   n_partials, (long)partial_stride, (const TT*)table, (long)table_stride, offset, ids, V, (TO*)out, n,
-                   dim, cols, status))));
+    const bool vec = dim % 4 == 0 && cols % 4 == 0 && z_stride % 4 == 0 && partial_stride % 4 == 0 && offset % 4 == 0 &&
+                     table_stride % 4 == 0 && (uintptr_t)z % 16 == 0 && (uintptr_t)table % 16 == 0 && (uintptr_t)out % 16 == 0;
+    const size_t total = (size_t)n * (vec ? cols / 4 : cols);
+    FB_DISPATCH_DTYPE(table_dtype, TT, FB_DISPATCH_DTYPE(out_dtype, TO, {
+        if (vec)
+            fb_launch((token_gate_kernel<TT, TO, 4>), (unsigned)((total + 255) / 256), 256, 0, stream, z, (long)z_stride,
+                      n_partials, (long)partial_stride, (const TT*)table, (long)table_stride, offset, ids, V, (TO*)out, n,
+                      dim, cols, status);
+        else
+            fb_launch((token_gate_kernel<TT, TO, 1>), (unsigned)((total + 255) / 256), 256, 0, stream, z, (long)z_stride,
+                      n_partials, (long)partial_stride, (const TT*)table, (long)table_stride, offset, ids, V, (TO*)out, n,
+                      dim, cols, status);
+    }));
     return fb_check_launch("token_gate");
 }

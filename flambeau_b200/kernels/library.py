@@ -67,7 +67,7 @@ _SIGNATURES = {
     "fb_moe_max_tiles": (I, [I, I, I]),
     "fb_moe_gather_rows": (I, [P, L, I, P, P, I, I, P, P, STREAM]),
     "fb_moe_sort": (I, [P, I, I, I, I, I, P, P, P, P, STREAM]),
-    "fb_moe_combine": (I, [P, L, P, P, I, P, I, L, P, P, I, I, P, I, L, STREAM]),
+    "fb_moe_combine": (I, [P, L, P, P, I, P, I, L, P, P, I, I, P, I, L, I, STREAM]),
     # layer_norm.cu
     "fb_add_layernorm": (I, [P, P, I, L, P, I, P, I, P, I, I, F, STREAM]),
     "fb_depth_average": (I, [P, P, I, L, P, L, I, P, I, L, STREAM]),

@@ -847,7 +847,8 @@ def paged_attention_mma(q, out, k_pool, v_pool, block_table, seq_q_start, seq_q_
         1 if any_short else 0,
         1 if any_long else 0, nh, nkv, hd, int(window), int(keep_first), float(scale), float(softcap),
         _slopes(score_slopes, nh), _ptr(sinks), *_head_gate(head_gate, q.shape[0], nh), 1 if weights_float32 else 0, scratch.data_ptr(), scratch.numel(),
-        *prefetch_arguments(prefetch), status.data_ptr(), _stream()), "paged_attention_mma", (n_seqs, nkv, hd))
+        *prefetch_arguments(prefetch), status.data_ptr(), _stream()), "paged_attention_mma",
+        (n_seqs, nkv, hd, "capped" if softcap > 0 else "head_gate" if head_gate is not None else ""))
 
 
 def attention_kv_share(nh: int, nkv: int) -> int:
@@ -1104,10 +1105,11 @@ def moe_sort(chosen, experts: int, tile: int, place_token, pair_place, tile_expe
 
 
 def moe_combine(expert_out, pair_place, share, shared_out, shared_partials: int, shared_partial_stride: int, gate,
-                out, n: int, pass_on=None) -> None:
+                out, n: int, pass_on=None, accumulate: bool = False) -> None:
     """out[t] = sum_k share[t, k] * expert_out[pair_place[t, k]] + gate[t] * sum of shared_out's shares (gate None:
     1).  pass_on ([n, D], optional): a pair without a place (an expert that has no weights) contributes
-    share * pass_on[t].  share None: every pair counts once (experts whose share scaled what they read)."""
+    share * pass_on[t].  share None: every pair counts once (experts whose share scaled what they read).  accumulate:
+    the sum is added to what `out` holds instead of replacing it."""
     _cuda(expert_out, pair_place, share, shared_out, gate, out, pass_on)
     if pass_on is not None and pass_on.shape[1] != out.shape[1]:
         raise KernelError("moe_combine: the rows handed on must have the output's width")
@@ -1121,7 +1123,7 @@ def moe_combine(expert_out, pair_place, share, shared_out, shared_partials: int,
                                _ptr(shared_out), int(shared_partials), int(shared_partial_stride), _ptr(gate),
                                out.data_ptr(), int(n), D, _ptr(pass_on),
                                dtype_code(pass_on) if pass_on is not None else 0,
-                               _rows(pass_on) if pass_on is not None else 0, _stream()), "moe_combine")
+                               _rows(pass_on) if pass_on is not None else 0, 1 if accumulate else 0, _stream()), "moe_combine")
 
 
 # ---------------------------------------------------------------------------

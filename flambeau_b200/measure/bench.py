@@ -33,6 +33,7 @@ size, decode and prefill tokens a second and the kernels that differ (flambeau_b
 `--only nodepel` likewise: the Nodepel design beside Mistral (flambeau_b200/measure/compare_nodepel.py; --sizes 1b,7b).
 `--only fegizen` likewise: the Fegizen design beside Nodepel (flambeau_b200/measure/compare_fegizen.py; --sizes 1b,7b).
 `--only tubepel` likewise: the Tubepel design beside Fegizen (flambeau_b200/measure/compare_tubepel.py; --sizes 1b,7b).
+`--only saropel` likewise: the Saropel design beside Tubepel (flambeau_b200/measure/compare_saropel.py; --sizes 1b,7b).
 
 The cache of the timed sequences is laid out by the cache manager exactly as a real request of that length
 leaves it (pages taken and, under the window, given back), but its keys and values are random numbers rather than
@@ -88,7 +89,8 @@ def main(argv=None) -> int:
     ap.add_argument("--layers", type=int, default=None, help="fewer layers than the shape has (sizes unchanged)")
     ap.add_argument("--prefill-tokens", type=int, default=2048)
     ap.add_argument("--skip-points", action="store_true", help="do not measure batch 1 and 64")
-    ap.add_argument("--only", choices=["all", "headline", "mixed", "shapes", "timeline", "mma-issue", "zedivik", "nodepel", "fegizen", "tubepel"],
+    ap.add_argument("--only", choices=["all", "headline", "mixed", "shapes", "timeline", "mma-issue", "zedivik", "nodepel", "fegizen", "tubepel",
+                                      "saropel"],
                     default="all",
                     help="headline: the shape's own line only; mixed / shapes: that part only; timeline: the kernels "
                          "of one decode step at --batch as the device ran them (a table on stderr, 4 layers unless "
@@ -217,6 +219,18 @@ def main(argv=None) -> int:
             result = compare_tubepel.run(sizes, args.layers or 4, args.batch, args.prefill_tokens, min(args.steps, 64),
                                          args.warmup, pk, gen, say)
         print(json.dumps({"impl": "ours", "metric": "Tubepel beside Fegizen at equal size: decode and prefill tok/s, "
+                          "per-kernel microseconds per launch", "dtype": "bf16", "data": "synthetic", "peak": tag,
+                          "peaks": {"hbm_gbs": pk["hbm_gbs"], "bf16_tflops": pk["bf16_tflops"]},
+                          "compare": result, "clocks": clocks.summary()}))
+        return 0
+    if args.only == "saropel":
+        from flambeau_b200.measure import compare_saropel
+        with ClockSampler(0) as clocks:
+            time.sleep(0.3)
+            sizes = [k for k in args.sizes.split(",") if k in compare_saropel.SIZES]
+            result = compare_saropel.run(sizes, args.layers or 4, args.batch, args.prefill_tokens, min(args.steps, 64),
+                                         args.warmup, pk, gen, say)
+        print(json.dumps({"impl": "ours", "metric": "Saropel beside Tubepel at equal size: decode and prefill tok/s, "
                           "per-kernel microseconds per launch", "dtype": "bf16", "data": "synthetic", "peak": tag,
                           "peaks": {"hbm_gbs": pk["hbm_gbs"], "bf16_tflops": pk["bf16_tflops"]},
                           "compare": result, "clocks": clocks.summary()}))

@@ -42,7 +42,7 @@ class RoutedExperts(FeedForward):
     a counting sort of the (token, choice) pairs into expert order
     with every expert's stretch padded to whole row tiles, two grouped products over that order (the first gathers
     the tokens' rows and applies the activation), and one kernel that brings the weighted outputs back to the
-    tokens and adds the shared expert.  All sizes on the host are upper bounds, so nothing is read back and the
+    tokens, adds the shared expert, and adds the sum to the stream where the block allows that.  All sizes on the host are upper bounds, so nothing is read back and the
     step can be replayed from a CUDA graph."""
     graph_safe = True
 
@@ -151,7 +151,7 @@ class RoutedExperts(FeedForward):
     def _shared_part(self, ctx, h, n):
         """The shared part's output: added to the stream by its own last product where that can be (None, 0, 0), else
         float32 shares in a buffer of its own (first share, how many, their stride)."""
-        kept = (ctx.delta_slabs, ctx.delta, ctx.pending_slabs, ctx.stream_x)
+        kept = (ctx.delta_slabs, ctx.delta, ctx.pending_slabs, getattr(ctx, "stream_x", None))
         sh = ctx.ws.alloc((ctx.max_slabs, n, self.width), torch.float32)
         ctx.delta_slabs, ctx.delta, ctx.pending_slabs = sh, sh[0], 1
         if self.token_gate:
@@ -210,9 +210,13 @@ class RoutedExperts(FeedForward):
                 shared, shared_stride = sh[0], sh.stride(0)
             elif self.shared is not None:
                 shared, shared_parts, shared_stride = self._shared_part(ctx, h, n)
+            # (where the block lets parts add to its stream, the sum joins it here and nothing is left to add)
+            stream = getattr(ctx, "stream_x", None)
+            to_stream = stream is not None
             ops.moe_combine(y, pair_place.view(n, K), None if self.share_on_input else share, shared, shared_parts,
-                            shared_stride, gate, out, n, pass_on=h[:n] if self.identity else None)
-        ctx.pending_slabs = 1
+                            shared_stride, gate, stream if to_stream else out, n,
+                            pass_on=h[:n] if self.identity else None, accumulate=to_stream)
+        ctx.pending_slabs = 0 if to_stream else 1
 
 
 register_part("feed_forward", "routed_experts", RoutedExperts)

@@ -156,7 +156,7 @@ def test_limited_experts_in_groups_with_a_gated_shared_expert(shape, dtype):
     from flambeau_b200.parts.spec import PartSpec
     n, D, E, K, ff, groups, shared = shape
     dt = DT[dtype]
-    b = Bench(dtype, max_step_tokens=1024, cache_tokens=1024)
+    b = Bench(dtype, max_step_tokens=1024, cache_tokens=2048)
     shared_spec = PartSpec("feed_forward", "gated_mlp", dict(width=D, inner=shared, activation="limited", limit=0.6, slope=1.702,
                                                              names=("gate", "up", "down")), "m.shared.") if shared else None
     count, keep = groups or (1, 0)
@@ -172,17 +172,18 @@ def test_limited_experts_in_groups_with_a_gated_shared_expert(shape, dtype):
     if groups:
         mlp["router"]["groups"] = {"count": count, "keep": keep}
     want = ps.routed_ff(h.double(), {k: v.double() for k, v in w.items()}, "m.", mlp)
-    ctx, x = b.begin([("a", [1] * n, [])], D)
-    x.zero_()
-    ctx.pending_slabs, ctx.stream_x = 1, x           # (the gated shared expert must not add itself to the stream)
-    part.forward(ctx, h.to(DEV), ctx.delta)
-    b.end()
-    assert float(x.abs().max()) == 0.0 and ctx.stream_x is x
-    out = ctx.delta_slabs[:ctx.pending_slabs].sum(0)
-    # a token whose choice was close may go to another expert in bfloat16: all but a few rows must agree
-    err = (out.double().cpu() - want).abs().max(dim=1).values / want.abs().max()
-    tol = 2e-5 if dtype == "float32" else 2e-2
-    assert int((err > tol).sum()) <= (0 if dtype == "float32" or K == E else n // 50), float(err.max())
+    for to_stream in (False, True):       # left for the next norm to add, or added to the block's stream by the part
+        ctx, x = b.begin([("a" if to_stream else "b", [1] * n, [])], D)
+        x.zero_()
+        ctx.pending_slabs, ctx.stream_x = 1, x if to_stream else None
+        part.forward(ctx, h.to(DEV), ctx.delta)
+        b.end()
+        assert ctx.pending_slabs == (0 if to_stream else 1) and (ctx.stream_x is x) == to_stream
+        out = x if to_stream else ctx.delta_slabs[:ctx.pending_slabs].sum(0)
+        # a token whose choice was close may go to another expert in bfloat16: all but a few rows must agree
+        err = (out.double().cpu() - want).abs().max(dim=1).values / want.abs().max()
+        tol = 2e-5 if dtype == "float32" else 2e-2
+        assert int((err > tol).sum()) <= (0 if dtype == "float32" or K == E else n // 50), float(err.max())
 
 
 GEOMETRIES = [(8, 2, 64, 64, 120, 16), (4, 2, 16, 24, 9, 16), (6, 1, 64, 64, 70, 16), (2, 2, 128, 128, 40, 32), (8, 4, 32, 32, 33, 8),
@@ -191,14 +192,14 @@ GEOMETRIES = [(8, 2, 64, 64, 120, 16), (4, 2, 16, 24, 9, 16), (6, 1, 64, 64, 70,
 
 
 @pytest.mark.parametrize("geometry", GEOMETRIES, ids=lambda g: "h%d-g%d-d%d-e%d-w%d-p%d" % g)
-@pytest.mark.parametrize("cap", [0.0, 3.0, 50.0])
+@pytest.mark.parametrize("cap", [0.0, 3.0, 50.0, 1000.0])
 @pytest.mark.parametrize("gated", [False, True], ids=["plain", "head-gate"])
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_attention_with_capped_scores_and_a_gate_per_head(geometry, cap, gated, dtype):
     """Over the paged cache, pages the window has passed given back and unreadable: first tokens, positions around the
     window's length, decoded tokens far into a request and at page borders, portions in mid-page and of two tokens.  The
     key at the window's far edge stands out along the query of head 0, the one just outside it more so.  A cap of 3
-    bends most scores of the standing-out keys, one of 50 hardly any."""
+    bends most scores of the standing-out keys, one of 50 hardly any; one of 1,000 takes the kernels' other form of the cap."""
     from flambeau_b200.kernels import ops
     nh, nkv, d, e, window, page = geometry
     dt = DT[dtype]
