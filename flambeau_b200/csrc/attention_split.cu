@@ -82,7 +82,7 @@ __device__ __forceinline__ void short_prefix(const AttnArgs& a, int G, const Sho
 // Adds the segments of one row of a pair: out = sum_c 2^(m_c - m) o_c / sum_c 2^(m_c - m) l_c, segments in slots
 // slot0 .. slot0 + n_chunks - 1.  One warp: a lane first takes a segment (its maximum, sum and weight), then a share
 // of the head's columns.  The partials were written by other SMs: they are read past the L1.
-template <int HD_MAX>
+template <int HD_MAX, bool EXTRA>
 __device__ __forceinline__ void merge_row(const AttnArgs& a, size_t slot0, int n_chunks, int r, int lane,
                                           __nv_bfloat16* dst, int row, int head) {
     constexpr int U = HD_MAX <= 128 ? 16 : 8;          // partials whose loads are in flight together
@@ -124,7 +124,7 @@ __device__ __forceinline__ void merge_row(const AttnArgs& a, size_t slot0, int n
         }
     }
     l = fb_warp_sum(l) + sink_term(a, head, m);
-    const float inv = (l > 0.0f ? 1.0f / l : 0.0f) * head_gate_factor(a, row, head);
+    const float inv = (l > 0.0f ? 1.0f / l : 0.0f) * (EXTRA ? head_gate_factor(a, row, head) : 1.0f);
 #pragma unroll
     for (int i = 0; i < HD_MAX / 32; ++i) {
         const int d = lane + 32 * i;
@@ -148,7 +148,8 @@ __host__ __device__ constexpr size_t split_smem_bytes(int hd_max, bool tma, size
            short_seqs_bytes(n_seqs) + 16;
 }
 
-template <int HD_MAX, bool TMA>
+// EXTRA: the launch caps its scores or gates its heads; without it neither costs the kernel a register.
+template <int HD_MAX, bool TMA, bool EXTRA>
 __global__ void __launch_bounds__(SPLIT_THREADS, HD_MAX <= 128 ? 2 : 1)
 attention_split_kernel(const __grid_constant__ AttnArgs a) {
     constexpr int NT = SPLIT_THREADS;
@@ -439,13 +440,13 @@ attention_split_kernel(const __grid_constant__ AttnArgs a) {
                     }
                 }
                 // ---- scale, mask, online softmax ----
-                const float to_log2 = a.cap_log2e > 0.0f ? 1.0f : a.scale_log2e;
-                if (a.cap_log2e > FB_SOFTCAP_DIRECT) {
+                const float to_log2 = EXTRA && a.cap_log2e > 0.0f ? 1.0f : a.scale_log2e;
+                if (EXTRA && a.cap_log2e > FB_SOFTCAP_DIRECT) {
 #pragma unroll
                     for (int nb = 0; nb < 2; ++nb)
 #pragma unroll
                         for (int e = 0; e < 4; ++e) s[nb][e] = fb_softcap(s[nb][e] * a.scale_over_cap, a.cap_log2e);
-                } else if (a.cap_log2e > 0.0f) {
+                } else if (EXTRA && a.cap_log2e > 0.0f) {
                     const float to_x = a.scale_over_cap * 2.8853900817779268f;
 #pragma unroll
                     for (int nb = 0; nb < 2; ++nb)
@@ -582,7 +583,7 @@ attention_split_kernel(const __grid_constant__ AttnArgs a) {
                     } else {                          // the whole pair was this CTA's: the result itself
                         const int token = q_start + r / G, head = kvh * G + r % G;
                         const float l_sink = l_all[h] + sink_term(a, head, m_all[h]);
-                        const float inv = (l_sink > 0.0f ? 1.0f / l_sink : 0.0f) * head_gate_factor(a, token, head);
+                        const float inv = (l_sink > 0.0f ? 1.0f / l_sink : 0.0f) * (EXTRA ? head_gate_factor(a, token, head) : 1.0f);
                         __nv_bfloat16* dst = a.out + (size_t)token * a.out_stride + (size_t)head * hd + 2 * (lane & 3);
 #pragma unroll
                         for (int d = 0; d < NDB; ++d) {
@@ -609,7 +610,7 @@ attention_split_kernel(const __grid_constant__ AttnArgs a) {
                 const size_t slot0 = (size_t)cur.c_first + pair;                     // consecutive CTAs, consecutive slots
                 for (int r = warp; r < rows_valid; r += SPLIT_SCORERS) {
                     const int token = q_start + r / G, head = kvh * G + r % G;
-                    merge_row<HD_MAX>(a, slot0, cur.n_chunks, r, lane,
+                    merge_row<HD_MAX, EXTRA>(a, slot0, cur.n_chunks, r, lane,
                                       a.out + (size_t)token * a.out_stride + (size_t)head * hd, token, head);
                 }
             }
@@ -621,9 +622,9 @@ attention_split_kernel(const __grid_constant__ AttnArgs a) {
 
 // Launches the split-key kernel with as many CTAs as are resident at once on this device (one equal stretch
 // each); fills in what depends on that number.
-template <int HD_MAX, bool TMA>
+template <int HD_MAX, bool TMA, bool EXTRA>
 int launch_split(AttnArgs& a, int n_seqs, long long scratch_floats, cudaStream_t stream) {
-    auto kern = attention_split_kernel<HD_MAX, TMA>;
+    auto kern = attention_split_kernel<HD_MAX, TMA, EXTRA>;
     static int per_sm = 0, per_sm_for = -1;
     static bool configured[FB_MAX_DEVICES] = {};
     const size_t smem = split_smem_bytes(HD_MAX, TMA, (size_t)n_seqs);
@@ -672,13 +673,15 @@ int fb_launch_attention_split(AttnArgs& a, int hd_max, bool tma, int n_seqs, flo
     FB_REQUIRE(n_seqs <= 1024, "attention_split: %d sequences in one step exceed 1024", n_seqs);
     a.n_seqs = n_seqs;
     a.part_o = scratch;
+    const bool extra = a.cap_log2e > 0.0f || a.head_gate;
+#define FB_SPLIT(HD_, TMA_)                                                                                           \
+    return extra ? launch_split<HD_, TMA_, true>(a, n_seqs, scratch_floats, stream)                                   \
+                 : launch_split<HD_, TMA_, false>(a, n_seqs, scratch_floats, stream)
     switch (hd_max) {
-        case 32: return launch_split<32, false>(a, n_seqs, scratch_floats, stream);
-        case 64: return tma ? launch_split<64, true>(a, n_seqs, scratch_floats, stream)
-                            : launch_split<64, false>(a, n_seqs, scratch_floats, stream);
-        case 128: return tma ? launch_split<128, true>(a, n_seqs, scratch_floats, stream)
-                             : launch_split<128, false>(a, n_seqs, scratch_floats, stream);
-        default: return tma ? launch_split<256, true>(a, n_seqs, scratch_floats, stream)
-                            : launch_split<256, false>(a, n_seqs, scratch_floats, stream);
+        case 32: FB_SPLIT(32, false);
+        case 64: if (tma) FB_SPLIT(64, true); else FB_SPLIT(64, false);
+        case 128: if (tma) FB_SPLIT(128, true); else FB_SPLIT(128, false);
+        default: if (tma) FB_SPLIT(256, true); else FB_SPLIT(256, false);
     }
+#undef FB_SPLIT
 }
