@@ -13,7 +13,10 @@ nothing), and given back
   * when a request ends, and
   * in a group with a window W, after the step that makes them dead: a page
     whose last position is below `length - W + 1` can be seen by no future
-    query (every future query sits at p >= length and sees [p-W+1, p]).
+    query (every future query sits at p >= length and sees [p-W+1, p]);
+  * in a group with chunks of C positions, after the step that fills a chunk: a
+    query sees its own chunk only, so the pages below the chunk that position
+    `length` lies in are dead.
 The reference bounds windowed layers with ring slabs instead and rejects paged
 windowed attention (crates/forward/src/core/composites/standard_attn.rs:436-441).
 
@@ -175,7 +178,10 @@ class CacheManager:
                     raise ValueError(f"call {ci} and call {plan.cache_from} disagree on the cache geometry")
                 # pages are given back by the owner's window: a reader that looks further back than the owner
                 # would ask for keys whose pages are gone
-                if plan.kv is not None and src.kv.release_window > 0 and (plan.kv.window == 0 or plan.kv.window > src.kv.window):
+                if plan.kv is not None and src.kv.chunk > 0 and plan.kv.chunk != src.kv.chunk:
+                    raise ValueError(f"call {ci} reads the cache of call {plan.cache_from}, which keeps chunks of "
+                                     f"{src.kv.chunk} keys, with chunks of {plan.kv.chunk or 'no'} keys")
+                if plan.kv is not None and src.kv.window > 0 and (plan.kv.window == 0 or plan.kv.window > src.kv.window):
                     raise ValueError(f"call {ci} reads the cache of call {plan.cache_from} with a window of "
                                      f"{plan.kv.window or 'all'} keys, but that cache keeps only {src.kv.window}")
                 continue
@@ -194,11 +200,13 @@ class CacheManager:
             if plan.state is not None:
                 sd = dtype if plan.state.dtype == "engine" else getattr(torch, plan.state.dtype)
                 self.state[ci] = torch.zeros((self.max_requests, *plan.state.shape), dtype=sd, device=device)
-        self.books = Books([g.n_pages for g in self.groups], [g.req.release_window for g in self.groups], self.page_size,
+        self.books = Books([g.n_pages for g in self.groups], [g.req.window for g in self.groups], self.page_size,
                            self.max_requests, self.max_pages_per_request,
-                           keep_first=[g.req.keep_first if g.req.release_window > 0 else 0 for g in self.groups])
+                           keep_first=[g.req.keep_first if g.req.window > 0 else 0 for g in self.groups],
+                           chunks=[g.req.chunk for g in self.groups])
         # Columns of a block-table row: the most live pages a request holds in any group.  A group with a window W
-        # keeps, while a step of k new tokens runs, the pages from position length - W + 1 to length + k.
+        # keeps, while a step of k new tokens runs, the pages from position length - W + 1 to length + k; one with
+        # chunks of C positions those from the start of length's chunk, at most C - 1 positions back.
         self.table_pages = 1
         for g in self.groups:
             live = self.max_pages_per_request

@@ -36,11 +36,12 @@ def _ptr(a: np.ndarray):
 
 
 class Books:
-    """One cache's books: `n_pages[g]` pages, window `windows[g]` (0 = none) and `keep_first[g]` first keys that stay
-    visible under the window (their pages are never given back while a request lives) for each group g."""
+    """One cache's books: `n_pages[g]` pages, window `windows[g]` (0 = none), `keep_first[g]` first keys that stay
+    visible under the window (their pages are never given back while a request lives) and chunk size `chunks[g]`
+    (0 = none: else a query sees the keys of its own chunk only) for each group g."""
 
     def __init__(self, n_pages: list, windows: list, page_size: int, max_requests: int, max_pages_per_request: int,
-                 keep_first: list | None = None):
+                 keep_first: list | None = None, chunks: list | None = None):
         if any(n <= 0 for n in n_pages):
             raise ValueError("a page pool needs at least one page")
         self._lib = lib()
@@ -49,6 +50,7 @@ class Books:
         self._h = self._lib.fbh_cache_new(self.n_groups, _ptr(_ints(n_pages if n_pages else [0])),
                                           _ptr(_ints(windows if windows else [0])),
                                           _ptr(_ints(keep_first if keep_first else [0] * max(self.n_groups, 1))),
+                                          _ptr(_ints(chunks if chunks else [0] * max(self.n_groups, 1))),
                                           int(page_size), int(max_requests), int(max_pages_per_request))
         if not self._h:
             raise PageError(self._message())

@@ -77,12 +77,14 @@ __device__ __forceinline__ float fb_gate_times(const FbGate& gate, float g, floa
 
 // ---- activations that stand alone ---------------------------------------------
 // out = act(z) for feed-forwards without a gate.  0 leaves z as it is.
-enum FbPlainAct : int { FB_PLAIN_NONE = 0, FB_PLAIN_SILU = 1, FB_PLAIN_GELU_TANH = 2, FB_PLAIN_RELU_SQUARED = 3 };
-inline bool fb_plain_act_known(int act) { return act >= FB_PLAIN_NONE && act <= FB_PLAIN_RELU_SQUARED; }
+enum FbPlainAct : int { FB_PLAIN_NONE = 0, FB_PLAIN_SILU = 1, FB_PLAIN_GELU_TANH = 2, FB_PLAIN_RELU_SQUARED = 3,
+                        FB_PLAIN_GELU = 4 };
+inline bool fb_plain_act_known(int act) { return act >= FB_PLAIN_NONE && act <= FB_PLAIN_GELU; }
 __device__ __forceinline__ float fb_plain_act(int act, float z) {
     if (act == FB_PLAIN_RELU_SQUARED) { const float r = fmaxf(z, 0.0f); return r * r; }
     if (act == FB_PLAIN_SILU) return z / (1.0f + expf(-z));
     if (act == FB_PLAIN_GELU_TANH) return fb_gelu_tanh(z);
+    if (act == FB_PLAIN_GELU) return 0.5f * z * (1.0f + erff(0.7071067811865476f * z));
     return z;
 }
 
@@ -153,6 +155,18 @@ __device__ __forceinline__ void fb_prefetch_issue(const FbPrefetch& pf, long wor
 // where the row has no column for the page (given back).
 __host__ __device__ __forceinline__ int fb_table_column(int logical, int base, int head) {
     return logical < head ? logical : (logical >= base ? logical - base + head : -1);
+}
+
+// ---- which keys a query sees -----------------------------------------------------
+// The first position that a query at position p sees under a window of the last `window` positions (0: none) and within
+// its own chunk of `chunk` positions, counted from position 0 (0: no chunks).  It never falls as p grows.
+__host__ __device__ __forceinline__ int fb_first_key(int p, int window, int chunk) {
+    int first = window > 0 && p - window + 1 > 0 ? p - window + 1 : 0;
+    if (chunk > 0) {
+        const int start = p / chunk * chunk;
+        if (start > first) first = start;
+    }
+    return first;
 }
 
 // ---- typed access -----------------------------------------------------------

@@ -4,6 +4,7 @@
 // keys live in the cache as [page][G][slot][2*kd] (both maps of a key/value head side by side) and values as
 // [page][G][slot][vd]; kd and vd are independent.  Per token and head:
 //     a_m = softmax_j(scale * q_m . k_m[j]) V        over the keys j in [max(0, p - W + 1), p]   (W = 0: all of [0, p])
+//                                                    and, with chunks of C positions, only those of p's own chunk
 //     o   = a_1 - lambda * a_2
 //     o  <- o / sqrt(mean(o^2) + eps) * out_scale * gate[token][h]            (gate optional)
 // Scores, softmax weights, the weighted sums, the difference and the norm are float32 whatever the storage type.
@@ -191,7 +192,7 @@ diff_attention_simt_kernel(const T* __restrict__ q, long q_stride, T* __restrict
                            int page_size, int n_pages, const int* __restrict__ block_table, int table_stride,
                            const int* __restrict__ table_base, const int* __restrict__ positions,
                            const int* __restrict__ row_seq, int n, int nh, int nkv, int kd, int vd, int window,
-                           float scale, float lambda, float eps, float out_scale, int* status) {
+                           int chunk, float scale, float lambda, float eps, float out_scale, int* status) {
     fb_pdl_launch_dependents();
     fb_pdl_wait();
     extern __shared__ float q_sh[];                    // [4 warps][2 * kd]
@@ -211,7 +212,7 @@ diff_attention_simt_kernel(const T* __restrict__ q, long q_stride, T* __restrict
     if (!active) return;
 
     const int p = positions[row];
-    const int t0 = (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
+    const int t0 = fb_first_key(p, window, chunk);
     const int* table = block_table + (size_t)row_seq[row] * table_stride;
     const int base_page = table_base ? table_base[row_seq[row]] : 0;
 
@@ -294,12 +295,12 @@ template <typename T, int NDR>
 static int launch_diff_simt(const void* q, long q_stride, void* out, long out_stride, const float* gate,
                             const void* k_pool, const void* v_pool, int page_size, int n_pages, const int* block_table,
                             int table_stride, const int* table_base, const int* positions, const int* row_seq, int n,
-                            int nh, int nkv, int kd, int vd, int window, float scale, float lambda, float eps,
+                            int nh, int nkv, int kd, int vd, int window, int chunk, float scale, float lambda, float eps,
                             float out_scale, int* status, cudaStream_t stream) {
     const long items = (long)n * nh;
     fb_launch((diff_attention_simt_kernel<T, NDR>), (unsigned)((items + 3) / 4), 128, 8 * kd * sizeof(float), stream,
               (const T*)q, q_stride, (T*)out, out_stride, gate, (const T*)k_pool, (const T*)v_pool, page_size, n_pages,
-              block_table, table_stride, table_base, positions, row_seq, n, nh, nkv, kd, vd, window, scale, lambda,
+              block_table, table_stride, table_base, positions, row_seq, n, nh, nkv, kd, vd, window, chunk, scale, lambda,
               eps, out_scale, status);
     return fb_check_launch("diff_attention_simt");
 }
@@ -308,17 +309,17 @@ FB_API int fb_diff_attention_simt(const void* q, long long q_stride, void* out, 
                                   const float* gate, const void* k_pool, const void* v_pool, int page_size,
                                   int n_pages, const int* block_table, int table_stride, const int* table_base,
                                   const int* positions, const int* row_seq, int n, int nh, int nkv, int kd, int vd,
-                                  int window, float scale, float lambda, float eps, float out_scale, int* status,
+                                  int window, int chunk, float scale, float lambda, float eps, float out_scale, int* status,
                                   cudaStream_t stream) {
     FB_REQUIRE(n >= 0 && nh > 0 && nkv > 0 && kd > 0 && vd > 0, "diff attention: bad sizes");
     FB_REQUIRE(nh % nkv == 0, "diff attention: %d query heads are not a multiple of %d key/value heads", nh, nkv);
     FB_REQUIRE(vd <= 512 && kd <= 1024, "diff attention: head sizes %d / %d are too large", kd, vd);
-    FB_REQUIRE(page_size > 0 && n_pages > 0 && window >= 0 && eps > 0.0f, "diff attention: bad cache geometry or eps");
+    FB_REQUIRE(page_size > 0 && n_pages > 0 && window >= 0 && chunk >= 0 && eps > 0.0f, "diff attention: bad cache geometry or eps");
     if (n == 0) return 0;
 #define FB_DIFF_CASE(NDR)                                                                                          \
     FB_DISPATCH_DTYPE(dtype, T, return (launch_diff_simt<T, NDR>(q, (long)q_stride, out, (long)out_stride, gate,   \
         k_pool, v_pool, page_size, n_pages, block_table, table_stride, table_base, positions, row_seq, n, nh, nkv, \
-        kd, vd, window, scale, lambda, eps, out_scale, status, stream)))
+        kd, vd, window, chunk, scale, lambda, eps, out_scale, status, stream)))
     if (vd <= 32) { FB_DIFF_CASE(1); }
     else if (vd <= 64) { FB_DIFF_CASE(2); }
     else if (vd <= 128) { FB_DIFF_CASE(4); }

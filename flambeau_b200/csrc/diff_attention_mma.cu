@@ -35,7 +35,7 @@ struct DiffArgs {
     int page_shift;                      // log2(page_size) where it is a power of two, else -1
     const int* block_table; int table_stride; const int* table_base;
     const int* seq_q_start; const int* seq_q_len; const int* seq_pos_start;
-    int n_seqs, nh, nkv, kd, vd, window;
+    int n_seqs, nh, nkv, kd, vd, window, chunk;
     float scale_log2e, lambda, eps, out_scale;
     int short_rows;                      // sequences with q_len * HG <= short_rows run in the split arrangement
     int n_splits;                        // split arrangement: CTAs per (sequence, key/value head)
@@ -95,9 +95,9 @@ diff_attention_mma_kernel(const DiffArgs a) {
     if (R0 >= rows_total) return;
     const int R1 = min(R0 + QROWS, rows_total) - 1;
     const int q_start = a.seq_q_start[seq], pos_start = a.seq_pos_start[seq];
-    const int kd = EXACT ? KSTEPS * 16 : a.kd, vd = EXACT ? VTILES * 8 : a.vd, W = a.window;
+    const int kd = EXACT ? KSTEPS * 16 : a.kd, vd = EXACT ? VTILES * 8 : a.vd;
     const int p_first = pos_start + R0 / HG, p_last = pos_start + R1 / HG;
-    const int t_lo = (W > 0 && p_first - W + 1 > 0) ? p_first - W + 1 : 0, t_hi = p_last;
+    const int t_lo = fb_first_key(p_first, a.window, a.chunk), t_hi = p_last;
     int tile_first = t_lo / KT, tile_last = t_hi / KT;
     if (SPLIT) {
         const int n_tiles = tile_last - tile_first + 1;
@@ -186,7 +186,7 @@ diff_attention_mma_kernel(const DiffArgs a) {
         const int R = R0 + row_tile * 16 + (lane >> 2) + 8 * i;
         row_ok[i] = R < rows_total;
         row_p[i] = pos_start + (row_ok[i] ? R : 0) / HG;
-        row_lo[i] = (W > 0 && row_p[i] - W + 1 > 0) ? row_p[i] - W + 1 : 0;
+        row_lo[i] = fb_first_key(row_p[i], a.window, a.chunk);
     }
 
     // byte addresses in shared memory of what this lane hands to ldmatrix: its row of Q, of a K tile (row = key,
@@ -206,12 +206,12 @@ diff_attention_mma_kernel(const DiffArgs a) {
     for (int vt = 0; vt < VTILES; ++vt) o[vt][0] = o[vt][1] = o[vt][2] = o[vt][3] = 0.0f;
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
 
-    // the warp's rows see every key of a tile when the tile lies between the last row's window start and the first
+    // the warp's rows see every key of a tile when the tile lies between the last row's first key and the first
     // row's position: such tiles need no mask
     const int warp_R0 = R0 + row_tile * 16;
     const bool warp_full = warp_R0 + 15 < rows_total;
     const int warp_p_min = pos_start + warp_R0 / HG;
-    const int warp_lo_max = W > 0 ? max(0, pos_start + min(warp_R0 + 15, rows_total - 1) / HG - W + 1) : 0;
+    const int warp_lo_max = fb_first_key(pos_start + min(warp_R0 + 15, rows_total - 1) / HG, a.window, a.chunk);
 
     // the stage of the tile in use and the stage to refill (the one tile kt-1 used), and their byte offsets, kept
     // as running values: NS is an argument, and a division per tile and thread is not free
@@ -556,12 +556,12 @@ FB_API int fb_diff_attention_mma(const void* q, long long q_stride, void* out, l
                                  const int* block_table, int table_stride, const int* table_base,
                                  const int* seq_q_start, const int* seq_q_len, const int* seq_pos_start, int n_seqs,
                                  int max_q_len, int any_short, int any_long, int nh, int nkv, int kd, int vd,
-                                 int window, float scale, float lambda, float eps, float out_scale, int n_splits,
+                                 int window, int chunk, float scale, float lambda, float eps, float out_scale, int n_splits,
                                  float* scratch, long long scratch_floats, int* status, cudaStream_t stream) {
     FB_REQUIRE(n_seqs >= 0 && nh > 0 && nkv > 0 && nh % nkv == 0, "diff attention: bad head counts");
     FB_REQUIRE(kd % 16 == 0 && kd >= 16 && kd <= 128, "diff attention (mma): key size %d is not a multiple of 16 up to 128", kd);
     FB_REQUIRE(vd % 16 == 0 && vd >= 16 && vd <= 256, "diff attention (mma): value size %d is not a multiple of 16 up to 256", vd);
-    FB_REQUIRE(page_size > 0 && n_pages > 0 && window >= 0 && eps > 0.0f, "diff attention: bad cache geometry or eps");
+    FB_REQUIRE(page_size > 0 && n_pages > 0 && window >= 0 && chunk >= 0 && eps > 0.0f, "diff attention: bad cache geometry or eps");
     FB_REQUIRE(scale > 0.0f, "diff attention (mma): the score scale must be positive");
     FB_REQUIRE(q_stride % 8 == 0 && out_stride % 2 == 0 && (uintptr_t)q % 16 == 0 && (uintptr_t)out % 4 == 0 &&
                (uintptr_t)k_pool % 16 == 0 && (uintptr_t)v_pool % 16 == 0, "diff attention (mma): unaligned operands");
@@ -577,7 +577,7 @@ FB_API int fb_diff_attention_mma(const void* q, long long q_stride, void* out, l
     for (int b = 0; b < 30; ++b) if ((1 << b) == page_size) a.page_shift = b;
     a.block_table = block_table; a.table_stride = table_stride; a.table_base = table_base;
     a.seq_q_start = seq_q_start; a.seq_q_len = seq_q_len; a.seq_pos_start = seq_pos_start;
-    a.n_seqs = n_seqs; a.nh = nh; a.nkv = nkv; a.kd = kd; a.vd = vd; a.window = window;
+    a.n_seqs = n_seqs; a.nh = nh; a.nkv = nkv; a.kd = kd; a.vd = vd; a.window = window; a.chunk = chunk;
     a.scale_log2e = scale * 1.4426950408889634f; a.lambda = lambda; a.eps = eps; a.out_scale = out_scale;
     a.short_rows = 16;
     a.n_splits = n_splits < 1 ? 1 : n_splits > 8 ? 8 : n_splits;

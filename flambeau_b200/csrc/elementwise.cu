@@ -885,6 +885,41 @@ FB_API int fb_sigmoid_gate(void* a, long long a_stride, int dtype, const float* 
 }
 
 // ---------------------------------------------------------------------------
+// x <- cap * tanh(x / cap) in place over float32 rows: the cap on a model's logits.
+// ---------------------------------------------------------------------------
+template <int VEC>
+__global__ void __launch_bounds__(256)
+softcap_rows_kernel(float* __restrict__ x, long stride, int n, int cols, float cap) {
+    fb_pdl_launch_dependents();
+    fb_pdl_wait();
+    const int per = cols / VEC;
+    const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (idx >= (size_t)n * per) return;
+    const int r = (int)(idx / per), c = (int)(idx - (size_t)r * per) * VEC;
+    float* p = x + (size_t)r * stride + c;
+    if constexpr (VEC == 4) {
+        float4 v = Vec4<float>::load(p);
+        v.x = cap * tanhf(v.x / cap); v.y = cap * tanhf(v.y / cap);
+        v.z = cap * tanhf(v.z / cap); v.w = cap * tanhf(v.w / cap);
+        Vec4<float>::store(p, v);
+    } else {
+        p[0] = cap * tanhf(p[0] / cap);
+    }
+}
+
+FB_API int fb_softcap_rows(float* x, long long stride, int n, int cols, float cap, cudaStream_t stream) {
+    FB_REQUIRE(n >= 0 && cols > 0 && stride >= cols && cap > 0.0f, "softcap_rows: bad arguments");
+    if (n == 0) return 0;
+    if (cols % 4 == 0 && stride % 4 == 0 && (uintptr_t)x % 16 == 0)
+        fb_launch(softcap_rows_kernel<4>, (unsigned)(((size_t)n * (cols / 4) + 255) / 256), 256, 0, stream, x, (long)stride, n,
+                  cols, cap);
+    else
+        fb_launch(softcap_rows_kernel<1>, (unsigned)(((size_t)n * cols + 255) / 256), 256, 0, stream, x, (long)stride, n, cols,
+                  cap);
+    return fb_check_launch("softcap_rows");
+}
+
+// ---------------------------------------------------------------------------
 // x[r, :] += v[:] for the first n rows of the float32 stream (a learned vector that joins every token alike), and
 // x[r, :] += y[r, :] of a second stream where there is one (added first).  Either may be absent.
 // ---------------------------------------------------------------------------

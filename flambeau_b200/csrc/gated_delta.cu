@@ -3,6 +3,8 @@
 //
 //     S <- g S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q        (g, beta: one number per head and token)
 //
+// or, with a decay per key channel, S <- diag(g) S with one number of g per row of S.
+//
 // Every column of S (one value dimension) goes through this on its own, so columns are spread over threads and a
 // request's tokens are taken in order; nothing but q, k, g and beta is shared between columns.
 //
@@ -10,20 +12,26 @@
 //   gdr_prepare      per (token, head of q, k or v): add the projection's split-K shares, the short causal convolution
 //                    over time with its SiLU (inputs before the portion's start come from the request's kept tail),
 //                    q and k made unit vectors per head (q also times `q_scale`), beta = sigmoid,
-//                    g = exp(-exp(A_log) * softplus(a + dt_bias)); all float32
+//                    g = exp(-exp(A_log) * softplus(a + dt_bias)) where a head has one; all float32 (decays per key
+//                    channel come from a map through a narrow middle: low_rank.cu)
 //   gdr_conv_tail    per request: the last taps-1 convolution inputs of the step become the kept tail
 //   gdr_recurrent    per (request, head, a few columns): the recurrence over the step's tokens, state in registers, 16
 //                    (or 32) lanes a column.  Both products with the state are taken from the state before the
 //                    token's update, a = S^T k and b = S^T q, so that they share one exchange between the lanes:
 //                    u = beta (v - g a), o = g b + u (k . q), S <- g S + k u^T, which is the same arithmetic; and two
 //                    tokens are taken at a time, the second one's products following from the first one's correction
-//   gdr_out_norm     per (token, head): o / rms(o) * weight * silu(gate), rounded to the engine's dtype
+//   gdr_channel_recurrent   the same recurrence with a decay per key channel.  Products are taken from the state as it
+//                    has decayed: with s = diag(g) S, a = s^T k and b = s^T q in one exchange, u = beta (v - a),
+//                    o = b + u (k . q), S <- s + k u^T; two tokens at a time, the second one's products from
+//                    diag(g') s plus the first one's correction times sum(g' k k') and sum(g' k q')
+//   gdr_out_norm     per (token, head): o / rms(o) * weight * act(gate) (silu, sigmoid, or the gate as it is), rounded to
+//                    the engine's dtype
 //
 // A request's slot of state is one float32 array: S as [heads][dv][dk] (a column's dk values side by side), then the
 // tail as [taps-1][channels]
-// (oldest first).  Projection rows are [q: G*dk | k: G*dk | v: H*dv | b: H | a: H | gate: H*dv]; head h of H reads
-// q/k head h / (H / G).
-#include "common.cuh"
+// (oldest first).  Projection rows begin [q: G*dk | k: G*dk | v: H*dv]; where beta, the decay and the gate lie behind
+// them are arguments; head h of H reads q/k head h / (H / G).
+#include "rows.cuh"
 
 __device__ __forceinline__ float gdr_slab_sum(const float* row, int c, int n_partials, long partial_stride) {
     float v = row[c];
@@ -36,8 +44,8 @@ __device__ __forceinline__ float gdr_softplus(float z) { return z > 20.0f ? z : 
 template <typename TW>
 __global__ void __launch_bounds__(128)
 gdr_prepare_kernel(const float* __restrict__ proj, long proj_stride, int n_partials, long partial_stride,
-                   const TW* __restrict__ conv_w, int taps, const TW* __restrict__ a_log, const TW* __restrict__ dt_bias,
-                   const float* __restrict__ state, long state_stride, long tail_off, const int* __restrict__ row_seq,
+                   const TW* __restrict__ conv_w, int taps, int b_off, int a_off, const TW* __restrict__ a_log,
+                   const TW* __restrict__ dt_bias, const float* __restrict__ state, long state_stride, long tail_off, const int* __restrict__ row_seq,
                    const int* __restrict__ seq_q_start, const int* __restrict__ seq_slot, float* __restrict__ qkv,
                    float* __restrict__ beta, float* __restrict__ decay, int G, int H, int dk, int dv, float q_scale,
                    float unit_eps) {
@@ -86,9 +94,10 @@ gdr_prepare_kernel(const float* __restrict__ proj, long proj_stride, int n_parti
     if (is_v && tid == 0) {
         const int h = unit - 2 * G;
         const float* pr = proj + (size_t)row * proj_stride;
-        const float b = gdr_slab_sum(pr, C + h, n_partials, partial_stride);
-        const float a = gdr_slab_sum(pr, C + H + h, n_partials, partial_stride);
+        const float b = gdr_slab_sum(pr, b_off + h, n_partials, partial_stride);
         beta[(size_t)row * H + h] = 1.0f / (1.0f + expf(-b));
+        if (!decay) return;
+        const float a = gdr_slab_sum(pr, a_off + h, n_partials, partial_stride);
         decay[(size_t)row * H + h] = expf(-expf(fb_to_float(a_log[h])) * gdr_softplus(a + fb_to_float(dt_bias[h])));
     }
 }
@@ -299,10 +308,225 @@ gdr_recurrent_kernel(const float* __restrict__ qkv, const float* __restrict__ be
     }
 }
 
+// ---------------------------------------------------------------------------
+// The recurrence with a decay per key channel.  A lane holds groups of four neighbouring key channels (R a multiple of 4:
+// they leave shared memory as 16-byte vectors and neighbouring lanes read neighbouring vectors), else every LPC-th.
+// ---------------------------------------------------------------------------
+template <int R, int LPC> struct GdcTile {
+    static constexpr int THREADS = 256, COLS = THREADS / LPC, DKP = LPC * R;
+    static constexpr int CH = DKP <= 128 ? 32 : DKP <= 256 ? 16 : 8;         // tokens fetched at a time, two such stages
+    static constexpr int STAGE_FLOATS = CH * (3 * DKP + COLS + 4);
+};
+
+__device__ __forceinline__ void gdr_copy16(float* dst, const float* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src)
+                 : "memory");
+}
+
+// BY4: rows of q, k, decay and the state start on 16-byte borders and dk is a multiple of 4.
+template <int R, int LPC, bool BY4>
+__global__ void __launch_bounds__(256)
+gdr_channel_recurrent_kernel(const float* __restrict__ qkv, const float* __restrict__ beta,
+                             const float* __restrict__ decay, float* __restrict__ state, long state_stride,
+                             const int* __restrict__ seq_q_start, const int* __restrict__ seq_q_len,
+                             const int* __restrict__ seq_slot, float* __restrict__ o, int G, int H, int dk, int dv) {
+    fb_pdl_launch_dependents();
+    fb_pdl_wait();
+    using Tile = GdcTile<R, LPC>;
+    constexpr int THREADS = Tile::THREADS, COLS = Tile::COLS, CH = Tile::CH, DKP = Tile::DKP;
+    constexpr bool VEC = R % 4 == 0;
+    extern __shared__ __align__(16) float sh[];
+    const int seq = blockIdx.x / H, head = blockIdx.x - seq * H;
+    const int g = head / (H / G);
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int li = tid % LPC, col = blockIdx.y * COLS + tid / LPC;
+    const bool live = col < dv;
+    const int qk = G * dk, C = 2 * qk + H * dv;
+    const int start = seq_q_start[seq], L = seq_q_len[seq];
+    float* S = state + (size_t)seq_slot[seq] * state_stride + ((size_t)head * dv + (live ? col : 0)) * dk;
+
+    // a stage: q, k, g [CH][DKP] each (rows padded with zeros beyond dk), v [CH][COLS], then [CH] each: beta, k_t . q_t,
+    // sum(g_t+1 k_t k_t+1), sum(g_t+1 k_t q_t+1)
+    auto fetch = [&](int t0, float* st) {
+        const int cnt = min(CH, L - t0);
+        float* qs = st;
+        float* ks = qs + CH * DKP;
+        float* gs = ks + CH * DKP;
+        float* vs = gs + CH * DKP;
+        constexpr int W = BY4 ? 4 : 1;
+        for (int e = tid * W; e < cnt * DKP; e += THREADS * W) {
+            const int t = e / DKP, d = e - t * DKP;
+            const size_t row = (size_t)(start + t0 + t);
+            if (d < dk) {
+                const float* rowp = qkv + row * C + (size_t)g * dk + d;
+                const float* gp = decay + (row * H + head) * dk + d;
+                if constexpr (BY4) {
+                    gdr_copy16(qs + e, rowp);
+                    gdr_copy16(ks + e, rowp + qk);
+                    gdr_copy16(gs + e, gp);
+                } else {
+                    gdr_copy4(qs + e, rowp);
+                    gdr_copy4(ks + e, rowp + qk);
+                    gdr_copy4(gs + e, gp);
+                }
+            } else {
+#pragma unroll
+                for (int u = 0; u < W; ++u) qs[e + u] = ks[e + u] = gs[e + u] = 0.0f;
+            }
+        }
+        for (int e = tid; e < cnt * COLS; e += THREADS) {
+            const int t = e / COLS, c2 = blockIdx.y * COLS + (e - t * COLS);
+            if (c2 < dv) gdr_copy4(vs + e, qkv + (size_t)(start + t0 + t) * C + 2 * qk + (size_t)head * dv + c2);
+            else vs[e] = 0.0f;
+        }
+        if (tid < cnt) gdr_copy4(vs + CH * COLS + tid, beta + (size_t)(start + t0 + tid) * H + head);
+        gdr_copies_commit();
+    };
+    auto channel = [&](int r) { return VEC ? (r / 4) * (4 * LPC) + 4 * li + (r & 3) : li + LPC * r; };
+    // this lane's channels of a row in shared memory
+    auto take = [&](const float* rowp, float (&out)[R]) {
+        if constexpr (VEC) {
+            const float4* p4 = reinterpret_cast<const float4*>(rowp) + li;
+#pragma unroll
+            for (int r = 0; r < R / 4; ++r) {
+                const float4 a = p4[r * LPC];
+                out[4 * r] = a.x; out[4 * r + 1] = a.y; out[4 * r + 2] = a.z; out[4 * r + 3] = a.w;
+            }
+        } else {
+#pragma unroll
+            for (int r = 0; r < R; ++r) out[r] = rowp[li + LPC * r];
+        }
+    };
+
+    float s[R];
+    if constexpr (BY4 && VEC) {
+#pragma unroll
+        for (int r = 0; r < R; r += 4) {
+            const int d = channel(r);
+            const float4 x = live && d < dk ? Vec4<float>::load(S + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+            s[r] = x.x; s[r + 1] = x.y; s[r + 2] = x.z; s[r + 3] = x.w;
+        }
+    } else {
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+            const int d = channel(r);
+            s[r] = (live && d < dk) ? S[d] : 0.0f;
+        }
+    }
+    if (L > 0) fetch(0, sh);
+    int buf = 0;
+    for (int t0 = 0; t0 < L; t0 += CH, buf ^= 1) {
+        const int cnt = min(CH, L - t0);
+        float* st = sh + buf * Tile::STAGE_FLOATS;
+        const bool more = t0 + CH < L;
+        if (more) fetch(t0 + CH, sh + (buf ^ 1) * Tile::STAGE_FLOATS);    // (its last readers passed the barrier below)
+        if (more) gdr_copies_wait<1>(); else gdr_copies_wait<0>();
+        __syncthreads();
+        const float* qs = st;
+        const float* ks = qs + CH * DKP;
+        const float* gs = ks + CH * DKP;
+        const float* vs = gs + CH * DKP;
+        const float* bs = vs + CH * COLS;
+        float* kq = st + CH * (3 * DKP + COLS + 1);
+        float* kgk = kq + CH;
+        float* kgq = kgk + CH;
+        for (int t = warp; t < cnt; t += THREADS / 32) {
+            const bool pair = !(t & 1) && t + 1 < cnt;
+            float acc = 0.0f, acc_k = 0.0f, acc_q = 0.0f;
+            for (int d = lane; d < DKP; d += 32) {
+                const float kd = ks[t * DKP + d];
+                acc = fmaf(kd, qs[t * DKP + d], acc);
+                if (pair) {
+                    const float gk = gs[(t + 1) * DKP + d] * kd;
+                    acc_k = fmaf(gk, ks[(t + 1) * DKP + d], acc_k);
+                    acc_q = fmaf(gk, qs[(t + 1) * DKP + d], acc_q);
+                }
+            }
+            acc = fb_warp_sum(acc);
+            acc_k = fb_warp_sum(acc_k);
+            acc_q = fb_warp_sum(acc_q);
+            if (lane == 0) { kq[t] = acc; kgk[t] = acc_k; kgq[t] = acc_q; }
+        }
+        __syncthreads();
+        int t = 0;
+        for (; t + 1 < cnt; t += 2) {
+            float k0[R], k1[R], x[R];
+            float a0 = 0.0f, b0 = 0.0f, a1 = 0.0f, b1 = 0.0f;
+            take(gs + t * DKP, x);
+#pragma unroll
+            for (int r = 0; r < R; ++r) s[r] *= x[r];
+            take(ks + t * DKP, k0);
+            take(qs + t * DKP, x);
+#pragma unroll
+            for (int r = 0; r < R; ++r) { a0 = fmaf(s[r], k0[r], a0); b0 = fmaf(s[r], x[r], b0); }
+            take(gs + (t + 1) * DKP, x);
+#pragma unroll
+            for (int r = 0; r < R; ++r) { s[r] *= x[r]; k0[r] *= x[r]; }
+            take(ks + (t + 1) * DKP, k1);
+            take(qs + (t + 1) * DKP, x);
+#pragma unroll
+            for (int r = 0; r < R; ++r) { a1 = fmaf(s[r], k1[r], a1); b1 = fmaf(s[r], x[r], b1); }
+#pragma unroll
+            for (int off = LPC / 2; off > 0; off >>= 1) {
+                a0 += __shfl_xor_sync(0xffffffffu, a0, off);
+                b0 += __shfl_xor_sync(0xffffffffu, b0, off);
+                a1 += __shfl_xor_sync(0xffffffffu, a1, off);
+                b1 += __shfl_xor_sync(0xffffffffu, b1, off);
+            }
+            const float u0 = bs[t] * (vs[t * COLS + tid / LPC] - a0);
+            const float u1 = bs[t + 1] * (vs[(t + 1) * COLS + tid / LPC] - fmaf(u0, kgk[t], a1));
+#pragma unroll
+            for (int r = 0; r < R; ++r) s[r] = fmaf(k1[r], u1, fmaf(k0[r], u0, s[r]));
+            if (live && li == 0) {
+                float* op = o + (size_t)(start + t0 + t) * H * dv + (size_t)head * dv + col;
+                op[0] = fmaf(u0, kq[t], b0);
+                op[(size_t)H * dv] = fmaf(u1, kq[t + 1], fmaf(u0, kgq[t], b1));
+            }
+        }
+        if (t < cnt) {                                 // the last token of an odd stretch
+            float k0[R], x[R];
+            float a = 0.0f, b = 0.0f;
+            take(gs + t * DKP, x);
+            take(ks + t * DKP, k0);
+#pragma unroll
+            for (int r = 0; r < R; ++r) { s[r] *= x[r]; a = fmaf(s[r], k0[r], a); }
+            take(qs + t * DKP, x);
+#pragma unroll
+            for (int r = 0; r < R; ++r) b = fmaf(s[r], x[r], b);
+#pragma unroll
+            for (int off = LPC / 2; off > 0; off >>= 1) {
+                a += __shfl_xor_sync(0xffffffffu, a, off);
+                b += __shfl_xor_sync(0xffffffffu, b, off);
+            }
+            const float u = bs[t] * (vs[t * COLS + tid / LPC] - a);
+#pragma unroll
+            for (int r = 0; r < R; ++r) s[r] = fmaf(k0[r], u, s[r]);
+            if (live && li == 0)
+                o[(size_t)(start + t0 + t) * H * dv + (size_t)head * dv + col] = fmaf(u, kq[t], b);
+        }
+        __syncthreads();                               // the stage may be overwritten by the fetch after next
+    }
+    if constexpr (BY4 && VEC) {
+#pragma unroll
+        for (int r = 0; r < R; r += 4) {
+            const int d = channel(r);
+            if (live && d < dk) Vec4<float>::store(S + d, make_float4(s[r], s[r + 1], s[r + 2], s[r + 3]));
+        }
+    } else {
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+            const int d = channel(r);
+            if (live && d < dk) S[d] = s[r];
+        }
+    }
+}
+
+enum FbGdrGate : int { FB_GDR_SILU = 0, FB_GDR_SIGMOID = 1, FB_GDR_AS_IS = 2 };
+
 template <typename TW, typename T>
 __global__ void __launch_bounds__(128)
 gdr_out_norm_kernel(const float* __restrict__ o, const float* __restrict__ proj, long proj_stride, int n_partials,
-                    long partial_stride, int gate_off, const TW* __restrict__ weight, float eps, T* __restrict__ out,
+                    long partial_stride, int gate_off, int gate_act, const TW* __restrict__ weight, float eps, T* __restrict__ out,
                     int n, int H, int dv) {
     fb_pdl_launch_dependents();
     fb_pdl_wait();
@@ -317,21 +541,26 @@ gdr_out_norm_kernel(const float* __restrict__ o, const float* __restrict__ proj,
     const float inv = 1.0f / sqrtf(s / (float)dv + eps);
     const float* pr = proj + (size_t)row * proj_stride;
     for (int d = lane; d < dv; d += 32) {
-        const float gate = gdr_slab_sum(pr, gate_off + head * dv + d, n_partials, partial_stride);
+        float gate = gdr_slab_sum(pr, gate_off + head * dv + d, n_partials, partial_stride);
+        if (gate_act == FB_GDR_SILU) gate = gdr_silu(gate);
+        else if (gate_act == FB_GDR_SIGMOID) gate = 1.0f / (1.0f + expf(-gate));
         out[(size_t)row * H * dv + (size_t)head * dv + d] =
-            fb_from_float<T>(x[d] * inv * fb_to_float(weight[d]) * gdr_silu(gate));
+            fb_from_float<T>(x[d] * inv * fb_to_float(weight[d]) * gate);
     }
 }
 
+// decay (with a_log, dt_bias and the columns from a_off on) may be null: no decay per head.
 FB_API int fb_gdr_prepare(const float* proj, long long proj_stride, int n_partials, long long partial_stride,
-                          const void* conv_w, int taps, const void* a_log, const void* dt_bias, int w_dtype,
+                          const void* conv_w, int taps, int b_off, int a_off, const void* a_log, const void* dt_bias, int w_dtype,
                           float* state, long long state_stride, long long tail_off, const int* row_seq,
                           const int* seq_q_start, const int* seq_q_len, const int* seq_slot, int n_seqs, float* qkv,
                           float* beta, float* decay, int n, int G, int H, int dk, int dv, float q_scale,
                           float unit_eps, cudaStream_t stream) {
     FB_REQUIRE(n >= 0 && G > 0 && H > 0 && H % G == 0 && dk > 0 && dv > 0 && taps >= 1, "gated delta: bad sizes");
     const long long C = 2LL * G * dk + (long long)H * dv;
-    FB_REQUIRE(proj_stride >= C + 2LL * H + (long long)H * dv, "gated delta: projection rows are too short");
+    FB_REQUIRE(b_off >= C && proj_stride >= (long long)b_off + H, "gated delta: projection rows are too short");
+    FB_REQUIRE(!decay || (a_log && dt_bias && a_off >= C && proj_stride >= (long long)a_off + H),
+               "gated delta: a decay per head wants its columns and parameters");
     if (n == 0) return 0;
     if (n_partials < 1) n_partials = 1;
     FB_REQUIRE(dk <= 1024 && dv <= 1024, "gated delta: head sizes up to 1024 (key %d, value %d)", dk, dv);
@@ -339,7 +568,7 @@ FB_API int fb_gdr_prepare(const float* proj, long long proj_stride, int n_partia
     FB_DISPATCH_DTYPE(w_dtype, TW, {
         auto kernel = gdr_prepare_kernel<TW>;
         fb_launch(kernel, dim3(n, 2 * G + H), dim3(128), 0, stream, proj, (long)proj_stride, n_partials, (long)partial_stride,
-                  (const TW*)conv_w, taps, (const TW*)a_log, (const TW*)dt_bias, (const float*)state, (long)state_stride,
+                  (const TW*)conv_w, taps, b_off, a_off, (const TW*)a_log, (const TW*)dt_bias, (const float*)state, (long)state_stride,
                   (long)tail_off, row_seq, seq_q_start, seq_slot, qkv, beta, decay, G, H, dk, dv, q_scale, unit_eps);
     });
     int rc = fb_check_launch("gdr_prepare");
@@ -383,16 +612,53 @@ FB_API int fb_gdr_recurrent(const float* qkv, const float* beta, const float* de
 #undef FB_GDR_CASE
 }
 
+template <int R, int LPC>
+static int launch_gdr_channel(const float* qkv, const float* beta, const float* decay, float* state, long state_stride,
+                              const int* seq_q_start, const int* seq_q_len, const int* seq_slot, int n_seqs, float* o,
+                              int G, int H, int dk, int dv, cudaStream_t stream) {
+    using Tile = GdcTile<R, LPC>;
+    const size_t smem = (size_t)2 * Tile::STAGE_FLOATS * sizeof(float);
+    const long C = 2L * G * dk + (long)H * dv;
+    const bool by4 = dk % 4 == 0 && C % 4 == 0 && state_stride % 4 == 0 && (uintptr_t)qkv % 16 == 0 &&
+                     (uintptr_t)decay % 16 == 0 && (uintptr_t)state % 16 == 0;
+    auto kernel = by4 ? gdr_channel_recurrent_kernel<R, LPC, true> : gdr_channel_recurrent_kernel<R, LPC, false>;
+    if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    fb_launch(kernel, dim3(n_seqs * H, (dv + Tile::COLS - 1) / Tile::COLS), dim3(Tile::THREADS), smem, stream, qkv, beta,
+              decay, state, state_stride, seq_q_start, seq_q_len, seq_slot, o, G, H, dk, dv);
+    return fb_check_launch("gdr_channel_recurrent");
+}
+
+// decay: float32 [rows][H][dk], one factor per head and key channel; the rest as in fb_gdr_recurrent.
+FB_API int fb_gdr_channel_recurrent(const float* qkv, const float* beta, const float* decay, float* state,
+                                    long long state_stride, const int* seq_q_start, const int* seq_q_len,
+                                    const int* seq_slot, int n_seqs, float* o, int G, int H, int dk, int dv,
+                                    cudaStream_t stream) {
+    FB_REQUIRE(n_seqs >= 0 && G > 0 && H > 0 && H % G == 0 && dk > 0 && dv > 0, "gated delta: bad sizes");
+    FB_REQUIRE(dk <= 1024, "gated delta: key size %d is larger than 1024", dk);
+    if (n_seqs == 0) return 0;
+#define FB_GDC_CASE(R, LPC) return launch_gdr_channel<R, LPC>(qkv, beta, decay, state, (long)state_stride, seq_q_start, \
+        seq_q_len, seq_slot, n_seqs, o, G, H, dk, dv, stream)
+    if (dk <= 16) FB_GDC_CASE(1, 16);
+    if (dk <= 32) FB_GDC_CASE(2, 16);
+    if (dk <= 64) FB_GDC_CASE(4, 16);
+    if (dk <= 128) FB_GDC_CASE(8, 16);
+    if (dk <= 256) FB_GDC_CASE(16, 16);
+    if (dk <= 512) FB_GDC_CASE(16, 32);
+    FB_GDC_CASE(32, 32);
+#undef FB_GDC_CASE
+}
+
 FB_API int fb_gdr_out_norm(const float* o, const float* proj, long long proj_stride, int n_partials,
-                           long long partial_stride, int gate_off, const void* weight, int w_dtype, float eps,
+                           long long partial_stride, int gate_off, int gate_act, const void* weight, int w_dtype, float eps,
                            void* out, int out_dtype, int n, int H, int dv, cudaStream_t stream) {
     FB_REQUIRE(n >= 0 && H > 0 && dv > 0, "gated delta: bad sizes");
+    FB_REQUIRE(gate_act >= FB_GDR_SILU && gate_act <= FB_GDR_AS_IS, "gated delta: unknown gate %d", gate_act);
     if (n == 0) return 0;
     if (n_partials < 1) n_partials = 1;
     const long items = (long)n * H;
     FB_DISPATCH_DTYPE(w_dtype, TW, FB_DISPATCH_DTYPE(out_dtype, T,
         (fb_launch((gdr_out_norm_kernel<TW, T>), dim3((unsigned)((items + 3) / 4)), dim3(128), 0, stream, o, proj,
-                   (long)proj_stride, n_partials, (long)partial_stride, gate_off, (const TW*)weight, eps, (T*)out, n, H,
+                   (long)proj_stride, n_partials, (long)partial_stride, gate_off, gate_act, (const TW*)weight, eps, (T*)out, n, H,
                    dv))));
     return fb_check_launch("gdr_out_norm");
 }

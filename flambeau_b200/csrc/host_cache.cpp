@@ -6,7 +6,8 @@
 // back (first in, first out), like the reference's host allocator
 // (crates/forward/src/core/scratch.rs:602-703); a request for several pages is all-or-nothing.  A page of a group
 // with a window W is given back after the step that makes it dead: a page whose last position is below
-// length - W + 1 can be seen by no future query.  The reference bounds windowed layers with ring slabs instead
+// length - W + 1 can be seen by no future query.  In a group whose queries see their own chunk of C positions only,
+// that holds for the pages below the chunk that position `length` lies in.  The reference bounds windowed layers with ring slabs instead
 // and rejects paged windowed attention (crates/forward/src/core/composites/standard_attn.rs:436-441); its
 // descriptor upload happens inside every layer (standard_attn.rs:315-329, 1133-1175).
 //
@@ -86,6 +87,7 @@ struct Cache {
     int page_size = 16, max_requests = 0, max_pages_per_request = 0;
     std::vector<Pool> pools;
     std::vector<int> windows;
+    std::vector<int> chunks;        // per group: queries see keys of their own chunk of this many positions (0: no chunks)
     std::vector<int> keep_pages;    // per group: pages that hold the first keys a window keeps visible (0 without)
     std::vector<Record> records;    // by slot
     std::vector<int> free_slots;    // a stack; the lowest slot on top at the start
@@ -108,10 +110,11 @@ int check_slot(const Cache& c, int slot) {
 
 FBH_API const char* fbh_last_error() { return g_error; }
 
-// n_pages[g], windows[g] (0 = all earlier keys stay live) and keep_first[g] (under a window: the first keys of a
-// request that stay visible, so the pages that hold them are kept; nullptr: none) per group.
-FBH_API void* fbh_cache_new(int n_groups, const int* n_pages, const int* windows, const int* keep_first, int page_size,
-                            int max_requests, int max_pages_per_request) {
+// n_pages[g], windows[g] (0 = all earlier keys stay live), keep_first[g] (under a window: the first keys of a
+// request that stay visible, so the pages that hold them are kept; nullptr: none) and chunks[g] (queries see the keys
+// of their own chunk of that many positions; nullptr or 0: no chunks) per group.
+FBH_API void* fbh_cache_new(int n_groups, const int* n_pages, const int* windows, const int* keep_first,
+                            const int* chunks, int page_size, int max_requests, int max_pages_per_request) {
     if (n_groups < 0 || page_size <= 0 || max_requests <= 0 || max_pages_per_request <= 0) {
         fail(ERR_STATE, "cache: bad geometry");
         return nullptr;
@@ -128,6 +131,7 @@ FBH_API void* fbh_cache_new(int n_groups, const int* n_pages, const int* windows
         }
         c->pools.emplace_back(n_pages[g]);
         c->windows.push_back(windows[g]);
+        c->chunks.push_back(chunks && chunks[g] > 0 ? chunks[g] : 0);
         const int keep = (keep_first && windows[g] > 0 && keep_first[g] > 0) ? keep_first[g] : 0;
         c->keep_pages.push_back((keep + page_size - 1) / page_size);
     }
@@ -292,9 +296,11 @@ FBH_API int fbh_commit(void* h, int n, const int* slots, const int* n_new) {
             return fail(ERR_STATE, "%d tokens committed, %d reserved", r.length + n_new[i], r.reserved_to);
         r.length += n_new[i];
         for (int g = 0; g < c.n_groups(); ++g) {
-            const int w = c.windows[(size_t)g];
-            if (w <= 0) continue;
-            const int first_live = r.length - w + 1;          // lowest position a future query can see
+            const int w = c.windows[(size_t)g], chunk = c.chunks[(size_t)g];
+            if (w <= 0 && chunk <= 0) continue;
+            // the lowest position a future query can see
+            int first_live = w > 0 ? r.length - w + 1 : 0;
+            if (chunk > 0 && r.length / chunk * chunk > first_live) first_live = r.length / chunk * chunk;
             PageList& pl = r.pages[(size_t)g];
             // logical pages [0, dead) are dead, but for the kept ones
             int dead = (first_live > 0 ? first_live : 0) / c.page_size;

@@ -12,7 +12,8 @@
 // Kernels:
 //   mla_latents   per token: the query's latent RMS-normed and rounded for the product that expands it; the
 //                 key/value latent RMS-normed, the shared key part rotated, both written into the token's cache row.
-//                 Inputs are the float32 split-K shares of the stacked down-projection.
+//                 Inputs are the float32 split-K shares of the stacked down-projection.  (A query without a latent of
+//                 its own, Rq = 0, needs nothing here: head_linear reads it from the shares.)
 //   head_linear   out[t, h, :N] = W_h [N, K] . a[t, h, :K] for every head, float32 accumulation on the CUDA cores;
 //                 `a` may be float32 shares (added first).  Two optional extras: K..K+r of the input row rotated into
 //                 N..N+r of the output row (the query side), and the result multiplied by sigmoid of a gate taken
@@ -44,7 +45,7 @@ mla_latents_kernel(const float* __restrict__ proj, long proj_stride, int n_parti
     __shared__ float red[32];
     const int t = blockIdx.x, tid = threadIdx.x;
     const float* pr = proj + (size_t)t * proj_stride;
-    if (blockIdx.y == 0) {                             // block-uniform
+    if (Rq > 0 && blockIdx.y == 0) {                   // block-uniform
         float ss = 0.0f;
         for (int i = tid; i < Rq; i += blockDim.x) {
             const float v = mla_slab_sum(pr, i, n_partials, partial_stride);
@@ -384,7 +385,7 @@ FB_API int fb_mla_latents(const float* proj, long long proj_stride, int n_partia
                           const float* cos_t, const float* sin_t, int half, int pairing, const int* positions,
                           const int* row_seq, const int* block_table, int table_stride, const int* table_base, void* pool, int out_dtype,
                           int page_size, int n_pages, int n, int* status, cudaStream_t stream) {
-    FB_REQUIRE(n >= 0 && Rq > 0 && Rc > 0 && r >= 0 && half >= 0 && 2 * half <= r, "latent attention: bad sizes");
+    FB_REQUIRE(n >= 0 && Rq >= 0 && (Rq > 0 ? wq && cq : pool != nullptr) && Rc > 0 && r >= 0 && half >= 0 && 2 * half <= r, "latent attention: bad sizes");
     FB_REQUIRE(eps > 0.0f, "latent attention: eps must be positive");
     FB_REQUIRE(half == 0 || (cos_t && sin_t), "latent attention: a rotation needs its tables");
     FB_REQUIRE(pairing == 0 || pairing == 1, "latent attention: pairs are neighbours (0) or halves (1)");
@@ -394,7 +395,7 @@ FB_API int fb_mla_latents(const float* proj, long long proj_stride, int n_partia
     const size_t smem = (size_t)(Rq > Rc ? Rq : Rc) * sizeof(float);
     FB_REQUIRE(smem <= 48 * 1024, "latent attention: a latent of more than 12288 numbers");
     FB_DISPATCH_DTYPE(w_dtype, TW, FB_DISPATCH_DTYPE(out_dtype, TO,
-        (fb_launch((mla_latents_kernel<TW, TO>), dim3(n, pool ? 2 : 1), dim3(256), smem, stream, proj, (long)proj_stride,
+        (fb_launch((mla_latents_kernel<TW, TO>), dim3(n, (Rq > 0 ? 1 : 0) + (pool ? 1 : 0)), dim3(256), smem, stream, proj, (long)proj_stride,
                    n_partials, (long)partial_stride, Rq, (const TW*)wq, (TO*)cq, kv_off, Rc, r, (const TW*)wkv, eps,
                    cos_t, sin_t, half, pairing, positions, row_seq, block_table, table_stride, table_base, (TO*)pool, page_size,
                    n_pages, status))));

@@ -1,17 +1,18 @@
 // A norm that takes the mean off first, with the residual add fused in front of it:
 //   r = rows ? rows[j] : j
-//   v = x[r] + sum_p delta[p][r]              (float32 slabs: a part's output, or the split-K shares of its last product)
-//   if (!rows && delta) x[r] = v              (the stream is updated in place)
+//   v = x[r] + sum_p delta[p][r] + bias       (float32 slabs: a part's output, or the split-K shares of its last product;
+//                                              bias: a vector that belongs to that product, optional)
+//   if (!rows && (delta || bias)) x[r] = v    (the stream is updated in place)
 //   out[j] = (v - mean(v)) / sqrt(mean((v - mean(v))^2) + eps) * w          (no bias)
 // Mean, deviations, their squares and the product with the weight are float32.  The row waits in shared memory
 // between the passes: the variance is taken from the deviations, not from the mean of squares, so that a row whose
 // mean is large against its spread keeps its digits.
-#include "common.cuh"
+#include "rows.cuh"
 
 template <typename TW, typename TO, bool VEC>
 __global__ void __launch_bounds__(1024)
 add_layernorm_kernel(float* __restrict__ x, const float* __restrict__ delta, int n_partials, size_t partial_stride,
-                     const TW* __restrict__ w, TO* __restrict__ out, const int* __restrict__ rows, int H, float eps) {
+                     const TW* __restrict__ bias, const TW* __restrict__ w, TO* __restrict__ out, const int* __restrict__ rows, int H, float eps) {
     fb_pdl_launch_dependents();
     fb_pdl_wait();
     extern __shared__ __align__(16) float ln_row[];
@@ -24,7 +25,11 @@ add_layernorm_kernel(float* __restrict__ x, const float* __restrict__ delta, int
         const int nvec = H >> 2;
         for (int c = threadIdx.x; c < nvec; c += blockDim.x) {
             float4 v = *reinterpret_cast<const float4*>(xr + 4 * c);
-            if (delta) {
+            if (delta || bias) {
+                if (bias) {
+                    const float4 b = Vec4<TW>::load(bias + 4 * c);
+                    v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
+                }
                 for (int p = 0; p < n_partials; ++p) {
                     const float4 d = *reinterpret_cast<const float4*>(delta + (size_t)p * partial_stride + (size_t)r * H + 4 * c);
                     v.x += d.x; v.y += d.y; v.z += d.z; v.w += d.w;
@@ -37,7 +42,8 @@ add_layernorm_kernel(float* __restrict__ x, const float* __restrict__ delta, int
     } else {
         for (int c = threadIdx.x; c < H; c += blockDim.x) {
             float v = xr[c];
-            if (delta) {
+            if (delta || bias) {
+                if (bias) v += fb_to_float(bias[c]);
                 for (int p = 0; p < n_partials; ++p) v += delta[(size_t)p * partial_stride + (size_t)r * H + c];
                 if (!rows) xr[c] = v;
             }
@@ -67,8 +73,9 @@ add_layernorm_kernel(float* __restrict__ x, const float* __restrict__ delta, int
     }
 }
 
-FB_API int fb_add_layernorm(float* x, const float* delta, int n_partials, long long partial_stride, const void* w,
-                            int w_dtype, void* out, int out_dtype, const int* rows, int n_out, int H, float eps,
+// bias (may be null) and w share a dtype.
+FB_API int fb_add_layernorm(float* x, const float* delta, int n_partials, long long partial_stride, const void* bias,
+                            const void* w, int w_dtype, void* out, int out_dtype, const int* rows, int n_out, int H, float eps,
                             cudaStream_t stream) {
     FB_REQUIRE(n_out >= 0 && H > 0, "add_layernorm: bad sizes n=%d H=%d", n_out, H);
     FB_REQUIRE(eps > 0.0f, "add_layernorm: eps must be positive");
@@ -77,7 +84,7 @@ FB_API int fb_add_layernorm(float* x, const float* delta, int n_partials, long l
     const size_t smem = (size_t)H * sizeof(float);
     FB_REQUIRE(smem <= 200 * 1024, "add_layernorm: width %d does not fit in shared memory", H);
     const bool vec = H % 4 == 0 && ((uintptr_t)x % 16 == 0) &&
-                     (!delta || ((uintptr_t)delta % 16 == 0 && partial_stride % 4 == 0));
+                     (uintptr_t)bias % 16 == 0 && (!delta || ((uintptr_t)delta % 16 == 0 && partial_stride % 4 == 0));
     const int per = vec ? H / 4 : H;
     const int threads = per >= 1024 ? 1024 : ((per + 31) / 32) * 32;
     FB_DISPATCH_DTYPE(w_dtype, TW, FB_DISPATCH_DTYPE(out_dtype, TO, {
@@ -85,12 +92,12 @@ FB_API int fb_add_layernorm(float* x, const float* delta, int n_partials, long l
             auto kernel = add_layernorm_kernel<TW, TO, true>;
             if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
             fb_launch(kernel, dim3(n_out), dim3(threads), smem, stream, x, delta, n_partials, (size_t)partial_stride,
-                      (const TW*)w, (TO*)out, rows, H, eps);
+                      (const TW*)bias, (const TW*)w, (TO*)out, rows, H, eps);
         } else {
             auto kernel = add_layernorm_kernel<TW, TO, false>;
             if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
             fb_launch(kernel, dim3(n_out), dim3(threads), smem, stream, x, delta, n_partials, (size_t)partial_stride,
-                      (const TW*)w, (TO*)out, rows, H, eps);
+                      (const TW*)bias, (const TW*)w, (TO*)out, rows, H, eps);
         }
     }));
     return fb_check_launch("add_layernorm");

@@ -7,7 +7,10 @@
 // size, a weight of that size), before the rotation in both cases.  The weight enters as (w + weight_offset).
 // Rotation: the first 2 * half dimensions of a head, dimension i paired with i + half, angles from the step's
 // cos/sin tables [n, half]; the rest of the head passes unchanged.  Value rows have a width of their own, and their
-// columns may be the keys' (`v_off`): the values are then the keys as projected, before norm and rotation.
+// columns may be the keys' (`v_off`): the values are then the keys as projected, before norm and rotation.  A bias over
+// the q, k and v columns (optional) joins the projection first.  `maps` neighbouring heads of q and of k may belong to
+// one head with several score maps: each is normalised and rotated alone, and a key's maps lie side by side in the
+// cache, whose key/value heads are then nkv / maps.
 //
 // Heads that are normalised alone (or not at all) and whose sizes are multiples of 4 go to a second kernel, one warp a
 // head: shares fetched 16 bytes at a time, the norm within the warp, the pairs exchanged through the warp's own stretch
@@ -25,23 +28,25 @@ __device__ __forceinline__ float qkr_slab_sum(const float* row, int c, int n_par
 template <typename TW, typename T>
 __global__ void __launch_bounds__(1024)
 qk_norm_rope_kv_write_kernel(const float* __restrict__ proj, long proj_stride, int n_partials, long partial_stride,
-                             const TW* __restrict__ q_weight, const TW* __restrict__ k_weight, int scope, float eps,
-                             float weight_offset, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
+                             const TW* __restrict__ bias, const TW* __restrict__ q_weight,
+                             const TW* __restrict__ k_weight, int scope, float eps, float weight_offset, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                              int half, T* __restrict__ q_out, long q_out_stride, const int* __restrict__ positions,
                              const int* __restrict__ row_seq, const int* __restrict__ block_table, int table_stride,
                              const int* __restrict__ table_base, int table_head, T* __restrict__ k_pool,
-                             T* __restrict__ v_pool, int page_size, int n_pages, int nh, int nkv, int hd, int vd,
-                             int v_off, int write_kv, int* status) {
+                             T* __restrict__ v_pool, int page_size, int n_pages, int nh, int nkv, int maps, int hd,
+                             int vd, int v_off, int write_kv, int* status) {
     fb_pdl_launch_dependents();
     fb_pdl_wait();
     extern __shared__ float sh[];                      // [qw + kw] the row's q and k; then one factor per head
     __shared__ float red[32];
     const int row = blockIdx.x, tid = threadIdx.x;
-    const int qw = nh * hd, kw = nkv * hd, vw = nkv * vd;
+    const int nv = nkv / maps;                         // key/value heads of the cache
+    const int qw = nh * hd, kw = nkv * hd, vw = nv * vd;
     const int heads = nh + nkv;
     float* inv = sh + qw + kw;                         // [heads]
     const float* pr = proj + (size_t)row * proj_stride;
-    for (int c = tid; c < qw + kw; c += blockDim.x) sh[c] = qkr_slab_sum(pr, c, n_partials, partial_stride);
+    for (int c = tid; c < qw + kw; c += blockDim.x)
+        sh[c] = qkr_slab_sum(pr, c, n_partials, partial_stride) + (bias ? fb_to_float(bias[c]) : 0.0f);
     __syncthreads();
     if (scope == FB_QK_NORM_PROJECTION) {
         float sq = 0.0f, sk = 0.0f;
@@ -76,8 +81,8 @@ qk_norm_rope_kv_write_kernel(const float* __restrict__ proj, long proj_stride, i
             if (tid == 0) atomicOr(status, FB_STATUS_BAD_PAGE);
         } else {
             // pools are [page][kv head][slot][row]: head g's row of this token
-            k_dst = k_pool + ((size_t)page * nkv * page_size + (p % page_size)) * hd;
-            v_dst = v_pool + ((size_t)page * nkv * page_size + (p % page_size)) * vd;
+            k_dst = k_pool + ((size_t)page * nv * page_size + (p % page_size)) * maps * hd;
+            v_dst = v_pool + ((size_t)page * nv * page_size + (p % page_size)) * vd;
         }
     }
     const float* cs = half ? cos_t + (size_t)row * half : nullptr;
@@ -105,20 +110,22 @@ qk_norm_rope_kv_write_kernel(const float* __restrict__ proj, long proj_stride, i
         if (is_q) {
             q_out[(size_t)row * q_out_stride + e] = fb_from_float<T>(y);
         } else if (k_dst) {
-            k_dst[(size_t)(h - nh) * page_size * hd + d] = fb_from_float<T>(y);
+            const int g = (h - nh) / maps, map = (h - nh) - g * maps;
+            k_dst[((size_t)g * page_size * maps + map) * hd + d] = fb_from_float<T>(y);
         }
     }
     if (v_dst) {
         for (int e = tid; e < vw; e += blockDim.x) {
             const int g = e / vd, d = e - g * vd;
             v_dst[(size_t)g * page_size * vd + d] =
-                fb_from_float<T>(qkr_slab_sum(pr, v_off + e, n_partials, partial_stride));
+                fb_from_float<T>(qkr_slab_sum(pr, v_off + e, n_partials, partial_stride) +
+                                 (bias ? fb_to_float(bias[v_off + e]) : 0.0f));
         }
     }
 }
 
-// A warp takes HPW neighbouring heads of a row: heads 0 .. nh - 1 are queries, the nkv behind them keys, the nkv behind
-// those values (none where the values are the keys as projected: the key's warp then writes both).  NV = float4 a lane
+// A warp takes HPW neighbouring heads of a row: heads 0 .. nh - 1 are queries, the nkv behind them keys, the nkv / maps
+// behind those values (none where the values are the keys as projected: the key's warp then writes both).  NV = float4 a lane
 // holds of a head.  Every load of the warp's heads is issued before the first use.  The two members of a rotated pair lie
 // 2 * half / 8 lanes apart where NV is 1 and half a multiple of 4 (one exchange between lanes); otherwise they meet in the
 // warp's stretch of shared memory.
@@ -126,17 +133,18 @@ constexpr int QKR_WARPS = 8;
 template <typename TW, typename T, int NV, int HPW>
 __global__ void __launch_bounds__(32 * QKR_WARPS)
 qk_norm_rope_heads_kernel(const float* __restrict__ proj, long proj_stride, int n_partials, long partial_stride,
-                          const TW* __restrict__ q_weight, const TW* __restrict__ k_weight, float eps,
-                          float weight_offset, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
+                          const TW* __restrict__ bias, const TW* __restrict__ q_weight,
+                          const TW* __restrict__ k_weight, float eps, float weight_offset, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                           int half, T* __restrict__ q_out, long q_out_stride, const int* __restrict__ positions,
                           const int* __restrict__ row_seq, const int* __restrict__ block_table, int table_stride,
                           const int* __restrict__ table_base, int table_head, T* __restrict__ k_pool,
-                          T* __restrict__ v_pool, int page_size, int n_pages, int n, int nh, int nkv, int hd, int vd,
-                          int v_off, int v_is_k, int write_kv, int* status) {
+                          T* __restrict__ v_pool, int page_size, int n_pages, int n, int nh, int nkv, int maps, int hd,
+                          int vd, int v_off, int v_is_k, int write_kv, int* status) {
     fb_pdl_launch_dependents();
     extern __shared__ float sh[];                      // [QKR_WARPS][hd], where pairs meet in shared memory
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int per_row = nh + (write_kv ? (v_is_k ? nkv : 2 * nkv) : 0);
+    const int nv = nkv / maps;                         // key/value heads of the cache
+    const int per_row = nh + (write_kv ? (v_is_k ? nkv : nkv + nv) : 0);
     const int groups = (per_row + HPW - 1) / HPW;
     const long item = (long)blockIdx.x * QKR_WARPS + warp;
     const int row = (int)(item / groups), h0 = (int)(item - (long)row * groups) * HPW;
@@ -187,7 +195,23 @@ qk_norm_rope_heads_kernel(const float* __restrict__ proj, long proj_stride, int 
         const int page = (entry >= 0 && entry < table_stride) ? block_table[(size_t)seq * table_stride + entry] : -1;
         cached = page >= 0 && page < n_pages;
         if (!cached && lane == 0) atomicOr(status, FB_STATUS_BAD_PAGE);
-        cache_row = (size_t)page * nkv * page_size + (p % page_size);
+        cache_row = (size_t)page * nv * page_size + (p % page_size);
+    }
+    if (bias) {
+#pragma unroll
+        for (int j = 0; j < HPW; ++j) {
+            const int h = h0 + j;
+            const bool is_v = h >= nh + nkv;
+            const int nvec = (is_v ? vd : hd) >> 2;
+            const TW* src = bias + (is_v ? v_off + (h - nh - nkv) * vd : h * hd);
+#pragma unroll
+            for (int i = 0; i < NV; ++i) {
+                const int c = lane + 32 * i;
+                if (h >= per_row || c >= nvec) continue;
+                const float4 b = Vec4<TW>::load(src + 4 * c);
+                x[j][i].x += b.x; x[j][i].y += b.y; x[j][i].z += b.z; x[j][i].w += b.w;
+            }
+        }
     }
     if (n_partials > 1) {
         // one head: its shares eight at a time; several: share after share, a load of every head in flight
@@ -218,7 +242,8 @@ qk_norm_rope_heads_kernel(const float* __restrict__ proj, long proj_stride, int 
         const int g = is_q ? h : is_v ? h - nh - nkv : h - nh;
         const int nvec = (is_v ? vd : hd) >> 2;
         if (!is_q && !cached) continue;
-        const size_t at = is_q ? 0 : cache_row + (size_t)g * page_size;
+        // the token's row in a pool (a key's maps share one)
+        const size_t at = is_q ? 0 : cache_row + (size_t)(is_v ? g : g / maps) * page_size;
         if (is_v || (!is_q && v_is_k)) {
             T* v_dst = v_pool + at * vd;
 #pragma unroll
@@ -275,7 +300,7 @@ qk_norm_rope_heads_kernel(const float* __restrict__ proj, long proj_stride, int 
                 }
             }
         }
-        T* dst = is_q ? q_out + (size_t)row * q_out_stride + (size_t)h * hd : k_pool + at * hd;
+        T* dst = is_q ? q_out + (size_t)row * q_out_stride + (size_t)h * hd : k_pool + (at * maps + g % maps) * hd;
 #pragma unroll
         for (int i = 0; i < NV; ++i) {
             const int c = lane + 32 * i;
@@ -284,14 +309,16 @@ qk_norm_rope_heads_kernel(const float* __restrict__ proj, long proj_stride, int 
     }
 }
 
-// proj: float32 rows [q: nh*hd | k: nkv*hd | ... v: nkv*vd from column v_off on ...], possibly as n_partials shares partial_stride elements apart.
+// proj: float32 rows [q: nh*hd | k: nkv*hd | ... v: nkv/maps*vd from column v_off on ...], possibly as n_partials shares
+// partial_stride elements apart.  bias (may be null): dtype w_dtype, by the same columns.  Pools: keys [page][nkv / maps]
+// [slot][maps * hd], values [page][nkv / maps][slot][vd].
 // q_weight / k_weight (dtype w_dtype): [hd] each for FB_QK_NORM_HEAD, [nh*hd] and [nkv*hd] for FB_QK_NORM_PROJECTION.
 FB_API int fb_qk_norm_rope_kv_write(const float* proj, long long proj_stride, int n_partials, long long partial_stride,
-                                    const void* q_weight, const void* k_weight, int w_dtype, int scope, float eps,
+                                    const void* bias, const void* q_weight, const void* k_weight, int w_dtype, int scope, float eps,
                                     float weight_offset, const float* cos_t, const float* sin_t, int half, void* q_out,
                                     long long q_out_stride, int out_dtype, const int* positions, const int* row_seq,
                                     const int* block_table, int table_stride, const int* table_base, int table_head,
-                                    void* k_pool, void* v_pool, int page_size, int n_pages, int n, int nh, int nkv, int hd, int vd,
+                                    void* k_pool, void* v_pool, int page_size, int n_pages, int n, int nh, int nkv, int maps, int hd, int vd,
                                     int v_off, int write_kv, int* status, cudaStream_t stream) {
     FB_REQUIRE(n >= 0 && nh > 0 && nkv > 0 && hd > 0 && vd > 0, "qk_norm_rope_kv_write: bad sizes");
     FB_REQUIRE(scope >= FB_QK_NORM_NONE && scope <= FB_QK_NORM_PROJECTION, "qk_norm_rope_kv_write: unknown reach %d", scope);
@@ -301,7 +328,10 @@ FB_API int fb_qk_norm_rope_kv_write(const float* proj, long long proj_stride, in
                "qk_norm_rope_kv_write: cache arguments missing");
     const int k_off = nh * hd;
     FB_REQUIRE(v_off >= k_off && (v_off != k_off || vd == hd), "qk_norm_rope_kv_write: values that are the keys have their size");
-    FB_REQUIRE(proj_stride >= (long long)(nh + nkv) * hd && proj_stride >= (long long)v_off + (long long)nkv * vd,
+    FB_REQUIRE(maps >= 1 && nkv % maps == 0 && (maps == 1 || v_off != k_off),
+               "qk_norm_rope_kv_write: %d key heads in maps of %d", nkv, maps);
+    const int nv = nkv / maps;
+    FB_REQUIRE(proj_stride >= (long long)(nh + nkv) * hd && proj_stride >= (long long)v_off + (long long)nv * vd,
                "qk_norm_rope_kv_write: projection rows are too short");
     if (n == 0) return 0;
     if (n_partials < 1) n_partials = 1;
@@ -311,12 +341,12 @@ FB_API int fb_qk_norm_rope_kv_write(const float* proj, long long proj_stride, in
     if (scope != FB_QK_NORM_PROJECTION && hd % 4 == 0 && vd % 4 == 0 && hd <= 512 && vd <= 512 && v_off % 4 == 0 &&
         proj_stride % 4 == 0 && partial_stride % 4 == 0 && q_out_stride % 4 == 0 && aligned(proj, 16) &&
         aligned(q_out, 4 * esize) && aligned(k_pool, 4 * esize) && aligned(v_pool, 4 * esize) &&
-        aligned(q_weight, 4 * wsize) && aligned(k_weight, 4 * wsize)) {
+        aligned(q_weight, 4 * wsize) && aligned(k_weight, 4 * wsize) && aligned(bias, 4 * wsize)) {
         if (scope == FB_QK_NORM_NONE) q_weight = k_weight = nullptr;
         const int v_is_k = v_off == k_off ? 1 : 0;
         // (a few rows: one head a warp, so that the heads spread over the device; a portion: four, for loads in flight)
         const int hpw = n <= 64 ? 1 : 4;
-        const int per_row = nh + (write_kv ? (v_is_k ? nkv : 2 * nkv) : 0);
+        const int per_row = nh + (write_kv ? (v_is_k ? nkv : nkv + nv) : 0);
         const long items = (long)n * ((per_row + hpw - 1) / hpw);
         const unsigned blocks = (unsigned)((items + QKR_WARPS - 1) / QKR_WARPS);
         const size_t smem_h = (size_t)QKR_WARPS * hd * sizeof(float);
@@ -324,9 +354,9 @@ FB_API int fb_qk_norm_rope_kv_write(const float* proj, long long proj_stride, in
 #define FB_QKR_HEADS(NV_, HPW_)                                                                                       \
         FB_DISPATCH_DTYPE(w_dtype, TW, FB_DISPATCH_DTYPE(out_dtype, T,                                                \
             (fb_launch((qk_norm_rope_heads_kernel<TW, T, NV_, HPW_>), dim3(blocks), dim3(32 * QKR_WARPS), smem_h, stream, \
-                       proj, (long)proj_stride, n_partials, (long)partial_stride, (const TW*)q_weight, (const TW*)k_weight, \
+                       proj, (long)proj_stride, n_partials, (long)partial_stride, (const TW*)bias, (const TW*)q_weight, (const TW*)k_weight, \
                        eps, weight_offset, cos_t, sin_t, half, (T*)q_out, (long)q_out_stride, positions, row_seq, block_table, \
-                       table_stride, table_base, table_head, (T*)k_pool, (T*)v_pool, page_size, n_pages, n, nh, nkv, hd, vd, \
+                       table_stride, table_base, table_head, (T*)k_pool, (T*)v_pool, page_size, n_pages, n, nh, nkv, maps, hd, vd, \
                        v_off, v_is_k, write_kv, status))))
         if (widest <= 128) { if (hpw == 1) FB_QKR_HEADS(1, 1); else FB_QKR_HEADS(1, 4); }
         else if (widest <= 256) { if (hpw == 1) FB_QKR_HEADS(2, 1); else FB_QKR_HEADS(2, 4); }
@@ -341,9 +371,9 @@ FB_API int fb_qk_norm_rope_kv_write(const float* proj, long long proj_stride, in
         if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         const int cols = (nh + 2 * nkv) * (hd > vd ? hd : vd);
         fb_launch(kernel, dim3(n), dim3(n > 128 ? 256 : cols >= 4096 ? 1024 : cols >= 1024 ? 512 : 256), smem, stream, proj, (long)proj_stride, n_partials, (long)partial_stride,
-                  (const TW*)q_weight, (const TW*)k_weight, scope, eps, weight_offset, cos_t, sin_t, half, (T*)q_out,
+                  (const TW*)bias, (const TW*)q_weight, (const TW*)k_weight, scope, eps, weight_offset, cos_t, sin_t, half, (T*)q_out,
                   (long)q_out_stride, positions, row_seq, block_table, table_stride, table_base, table_head, (T*)k_pool,
-                  (T*)v_pool, page_size, n_pages, nh, nkv, hd, vd, v_off, write_kv, status);
+                  (T*)v_pool, page_size, n_pages, nh, nkv, maps, hd, vd, v_off, write_kv, status);
     }));
     return fb_check_launch("qk_norm_rope_kv_write");
 }

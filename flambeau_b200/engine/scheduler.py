@@ -171,8 +171,8 @@ class Scheduler:
                 self._preempt(victim, plan)
 
     def _pages_for(self, tokens: int, group: int) -> int:
-        """Pages that `tokens` tokens of one request hold in a group at most (a window keeps the last W tokens,
-        plus the portion that is being written and the page the window starts in)."""
+        """Pages that `tokens` tokens of one request hold in a group at most (a window keeps the last W tokens, a
+        chunk at most its own, plus the portion that is being written and the page the window or the chunk starts in)."""
         req = self.cache.groups[group].req
         window = req.release_window
         page = self.cache.page_size

@@ -48,6 +48,8 @@ class StepContext:
         self.max_slabs = 1                  # how many split-K slabs a product may leave for the next kernel to add
         self.pending_slabs = 1
         self.stream_x = None                # the residual stream of the block that is running (set by the block)
+        self.bias_can_wait = False          # the block's next norm adds the bias of a part's last product (set by the block)
+        self.pending_bias = None            # that bias
         self.l2_hints = engine.l2_hints
 
     def open_stream(self, width: int):
@@ -66,14 +68,22 @@ class StepContext:
         self.pending_slabs = 1
         return x
 
-    def to_stream(self, linear, a) -> None:
+    def to_stream(self, linear, a, bias=None) -> None:
         """The last product of a mixer or a feed-forward, whose result belongs on the residual stream: added to
         the stream by the product's own epilogue where that is possible (ctx.pending_slabs = 0: nothing is left to
-        add), else left in ctx.delta_slabs for the next norm to add (ctx.pending_slabs = how many slabs)."""
+        add), else left in ctx.delta_slabs for the next norm to add (ctx.pending_slabs = how many slabs).  `bias` (a
+        vector that belongs to the product) is left to that norm too where it takes one (ctx.pending_bias), else added
+        by a kernel of its own."""
         if self.stream_x is not None and linear.add_into(self, a, self.stream_x):
             self.pending_slabs = 0
         else:
             self.pending_slabs = linear.slabs(self, a, self.delta_slabs)
+        if bias is None:
+            return
+        if self.bias_can_wait:
+            self.pending_bias = bias
+        else:
+            ops.add_row(self.stream_x if self.pending_slabs == 0 else self.delta, bias)
 
     def step_alloc(self, shape, dtype):
         """Scratch that lives until the step ends (ctx.ws allocations end with their scope)."""

@@ -34,6 +34,7 @@ _SIGNATURES = {
     "fb_rope_kv_write": (I, [P, L, I, L, P, L, P, L, P, L, I, I, P, P, I, P, P, P, I, P, I, P, P, I, I, I, I, I, I, I, P, STREAM]),
     "fb_gate_mul": (I, [P, L, I, I, L, P, I, I, I, I, F, F, STREAM]),
     "fb_activation": (I, [P, L, I, I, L, P, I, I, I, I, STREAM]),
+    "fb_softcap_rows": (I, [P, L, I, I, F, STREAM]),
     "fb_add_row": (I, [P, P, P, I, I, I, STREAM]),
     "fb_add_slabs": (I, [P, P, I, L, P, I, I, I, STREAM]),
     "fb_sigmoid_gate": (I, [P, L, I, P, L, I, L, I, I, STREAM]),
@@ -56,12 +57,15 @@ _SIGNATURES = {
     # attention_simt.cu
     "fb_paged_attention_simt": (I, [P, L, P, L, I, P, P, I, I, P, I, P, I, P, P, I, I, I, I, I, I, I, F, F, P, P, P, L, I, L, P, STREAM]),
     # qk_norm_rope.cu
-    "fb_qk_norm_rope_kv_write": (I, [P, L, I, L, P, P, I, I, F, F, P, P, I, P, L, I, P, P, P, I, P, I, P, P, I, I, I, I,
-                                     I, I, I, I, I, P, STREAM]),
+    "fb_qk_norm_rope_kv_write": (I, [P, L, I, L, P, P, P, I, I, F, F, P, P, I, P, L, I, P, P, P, I, P, I, P, P, I, I, I, I,
+                                     I, I, I, I, I, I, P, STREAM]),
     # gated_delta.cu
-    "fb_gdr_prepare": (I, [P, L, I, L, P, I, P, P, I, P, L, L, P, P, P, P, I, P, P, P, I, I, I, I, I, F, F, STREAM]),
+    "fb_gdr_prepare": (I, [P, L, I, L, P, I, I, I, P, P, I, P, L, L, P, P, P, P, I, P, P, P, I, I, I, I, I, F, F, STREAM]),
     "fb_gdr_recurrent": (I, [P, P, P, P, L, P, P, P, I, P, I, I, I, I, STREAM]),
-    "fb_gdr_out_norm": (I, [P, P, L, I, L, I, P, I, F, P, I, I, I, I, STREAM]),
+    "fb_gdr_channel_recurrent": (I, [P, P, P, P, L, P, P, P, I, P, I, I, I, I, STREAM]),
+    "fb_gdr_out_norm": (I, [P, P, L, I, L, I, I, P, I, F, P, I, I, I, I, STREAM]),
+    # low_rank.cu
+    "fb_low_rank_maps": (I, [P, L, I, L, I, I, P, I, P, P, P, P, P, P, P, P, STREAM]),
     # moe.cu
     "fb_moe_choose": (I, [P, L, I, L, P, I, I, I, I, I, P, P, P, I, F, I, I, I, STREAM]),
     "fb_moe_max_tiles": (I, [I, I, I]),
@@ -69,7 +73,7 @@ _SIGNATURES = {
     "fb_moe_sort": (I, [P, I, I, I, I, I, P, P, P, P, STREAM]),
     "fb_moe_combine": (I, [P, L, P, P, I, P, I, L, P, P, I, I, P, I, L, I, STREAM]),
     # layer_norm.cu
-    "fb_add_layernorm": (I, [P, P, I, L, P, I, P, I, P, I, I, F, STREAM]),
+    "fb_add_layernorm": (I, [P, P, I, L, P, P, I, P, I, P, I, I, F, STREAM]),
     "fb_depth_average": (I, [P, P, I, L, P, L, I, P, I, L, STREAM]),
     # time_conv.cu
     "fb_time_conv": (I, [P, P, I, P, L, L, P, P, P, P, I, P, I, I, I, STREAM]),
@@ -83,12 +87,12 @@ _SIGNATURES = {
     # diff_attention.cu
     "fb_qkv_bias_cache_write": (I, [P, L, I, L, P, I, P, L, I, P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, I, P,
                                     STREAM]),
-    "fb_diff_attention_simt": (I, [P, L, P, L, I, P, P, P, I, I, P, I, P, P, P, I, I, I, I, I, I, F, F, F, F, P,
+    "fb_diff_attention_simt": (I, [P, L, P, L, I, P, P, P, I, I, P, I, P, P, P, I, I, I, I, I, I, I, F, F, F, F, P,
                                    STREAM]),
     # diff_attention_mma.cu
     "fb_diff_attention_scratch_floats": (L, [I, I, I, I]),
     "fb_diff_attention_splits": (I, [I, I, I, I, I]),
-    "fb_diff_attention_mma": (I, [P, L, P, L, P, P, P, I, I, P, I, P, P, P, P, I, I, I, I, I, I, I, I, I, F, F, F, F, I,
+    "fb_diff_attention_mma": (I, [P, L, P, L, P, P, P, I, I, P, I, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, F, F, F, I,
                                   P, L, P, STREAM]),
     # attention_mma.cu
     "fb_paged_attention_mma": (I, [P, L, P, L, P, P, I, I, P, I, P, I, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, F, P, P,
@@ -99,7 +103,7 @@ _SIGNATURES = {
     "fb_sample": (I, [P, L, I, I, P, P, P, P, P, P, STREAM]),
     # host side of the cache manager and of a step's descriptor (csrc/host_cache.cpp)
     "fbh_last_error": (c_char_p, []),
-    "fbh_cache_new": (P, [I, P, P, P, I, I, I]),
+    "fbh_cache_new": (P, [I, P, P, P, P, I, I, I]),
     "fbh_cache_free": (None, [P]),
     "fbh_has_slot": (I, [P]),
     "fbh_admit": (I, [P]),

@@ -177,9 +177,10 @@ def qkv_bias_cache_write(proj: torch.Tensor, bias, q_out: torch.Tensor, gate_out
 
 
 def diff_attention_simt(q, out, gate, cache, positions, row_seq, nh: int, nkv: int, kd: int, vd: int, window: int,
-                        scale: float, lam: float, eps: float, out_scale: float, status) -> None:
+                        scale: float, lam: float, eps: float, out_scale: float, status, chunk: int = 0) -> None:
     """Differential attention with float32 math on the CUDA cores (see csrc/diff_attention.cu): q [n, nh*2*kd],
-    out [n, nh*vd], gate float32 [n, nh] or None."""
+    out [n, nh*vd], gate float32 [n, nh] or None.  chunk > 0: a query sees the keys of its own chunk of that many
+    positions, counted from position 0."""
     _cuda(q, out, gate, positions, row_seq, status)
     n = q.shape[0]
     k_pool, v_pool = cache.k_pool, cache.v_pool
@@ -194,7 +195,7 @@ def diff_attention_simt(q, out, gate, cache, positions, row_seq, nh: int, nkv: i
     check(lib().fb_diff_attention_simt(
         q.data_ptr(), _rows(q), out.data_ptr(), _rows(out), dtype_code(q), _ptr(gate), k_pool.data_ptr(),
         v_pool.data_ptr(), cache.page_size, n_pages, cache.block_table.data_ptr(), cache.block_table.stride(0),
-        _ptr(cache.table_base), positions.data_ptr(), row_seq.data_ptr(), n, nh, nkv, kd, vd, int(window),
+        _ptr(cache.table_base), positions.data_ptr(), row_seq.data_ptr(), n, nh, nkv, kd, vd, int(window), int(chunk),
         float(scale), float(lam), float(eps), float(out_scale), status.data_ptr(), _stream()), "diff_attention_simt")
 
 
@@ -285,7 +286,7 @@ def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, n_partials: int = 1, part
     gate_mul(gate_up, out, n_partials, partial_stride, "silu")
 
 
-PLAIN_ACTIVATIONS = {None: 0, "none": 0, "silu": 1, "gelu_tanh": 2, "relu_squared": 3}   # activations without a gate
+PLAIN_ACTIVATIONS = {None: 0, "none": 0, "silu": 1, "gelu_tanh": 2, "relu_squared": 3, "gelu": 4}   # activations without a gate
 
 
 def plain_activation_code(name) -> int:
@@ -304,6 +305,14 @@ def activation(z: torch.Tensor, out: torch.Tensor, name: str, n_partials: int = 
     check(lib().fb_activation(z.data_ptr(), _rows(z), dtype_code(z), int(n_partials), int(partial_stride),
                               out.data_ptr(), dtype_code(out), n, I, plain_activation_code(name), _stream()),
           "activation")
+
+
+def softcap_rows(x: torch.Tensor, cap: float) -> None:
+    """x <- cap * tanh(x / cap) in place; float32 rows."""
+    _cuda(x)
+    if x.dtype != torch.float32:
+        raise KernelError("softcap_rows: float32 rows wanted")
+    check(lib().fb_softcap_rows(x.data_ptr(), _rows(x), x.shape[0], x.shape[1], float(cap), _stream()), "softcap_rows")
 
 
 def add_row(x: torch.Tensor, v, y=None) -> None:
@@ -899,11 +908,13 @@ def diff_attention_mma_supported(q: torch.Tensor, nh: int, nkv: int, kd: int, vd
 
 def diff_attention_mma(q, out, gate, cache, seq_q_start, seq_q_len, seq_pos_start, n_seqs: int, max_q_len: int,
                        max_kv_len: int, any_short: bool, any_long: bool, nh: int, nkv: int, kd: int, vd: int,
-                       window: int, scale: float, lam: float, eps: float, out_scale: float, status, alloc=None) -> None:
+                       window: int, scale: float, lam: float, eps: float, out_scale: float, status, alloc=None,
+                       chunk: int = 0) -> None:
     """Differential attention on the tensor cores (csrc/diff_attention_mma.cu).  Sequences are described per entry of
     the step (first row, rows, first position); any_short / any_long say whether the step holds sequences with
     rows * (nh / nkv) <= 16 / > 16, which run in the split-key and in the portion arrangement.  `alloc(n)` returns
-    n float32 of scratch for the split arrangement's partials (default: a fresh tensor)."""
+    n float32 of scratch for the split arrangement's partials (default: a fresh tensor).  chunk: see
+    diff_attention_simt."""
     _cuda(q, out, gate, seq_q_start, seq_q_len, seq_pos_start, status)
     k_pool, v_pool = cache.k_pool, cache.v_pool
     n_pages = k_pool.shape[0]
@@ -919,7 +930,7 @@ def diff_attention_mma(q, out, gate, cache, seq_q_start, seq_q_len, seq_pos_star
         raise KernelError("diff attention: the gate wants contiguous float32 [n, heads]")
     splits, scratch = 1, None
     if any_short:
-        max_keys = min(max_kv_len, window + 16) if window > 0 else max_kv_len
+        max_keys = min([max_kv_len] + [n + 16 for n in (window, chunk) if n > 0])
         splits = lib().fb_diff_attention_splits(n_seqs, nkv, max(1, int(max_keys)), kd, vd)
         floats = lib().fb_diff_attention_scratch_floats(n_seqs, nkv, vd, splits)
         scratch = alloc(floats) if alloc is not None else torch.empty(floats, dtype=torch.float32, device=q.device)
@@ -927,13 +938,13 @@ def diff_attention_mma(q, out, gate, cache, seq_q_start, seq_q_len, seq_pos_star
         q.data_ptr(), _rows(q), out.data_ptr(), _rows(out), _ptr(gate), k_pool.data_ptr(), v_pool.data_ptr(),
         cache.page_size, n_pages, cache.block_table.data_ptr(), cache.block_table.stride(0), _ptr(cache.table_base),
         seq_q_start.data_ptr(), seq_q_len.data_ptr(), seq_pos_start.data_ptr(), n_seqs, max_q_len,
-        1 if any_short else 0, 1 if any_long else 0, nh, nkv, kd, vd, int(window), float(scale), float(lam),
+        1 if any_short else 0, 1 if any_long else 0, nh, nkv, kd, vd, int(window), int(chunk), float(scale), float(lam),
         float(eps), float(out_scale), splits, _ptr(scratch), scratch.numel() if scratch is not None else 0,
         status.data_ptr(), _stream()), "diff_attention_mma")
 
 
 def diff_attention(ctx, q, out, gate, cache, nh: int, nkv: int, kd: int, vd: int, window: int, scale: float,
-                   lam: float, eps: float, out_scale: float) -> None:
+                   lam: float, eps: float, out_scale: float, chunk: int = 0) -> None:
     """Differential attention of every row of the step over its request's cached keys and values, with the kernel
     that fits the dtype and the sizes: the tensor-core arrangements for bfloat16 and sizes they take, the
     float32-math kernel otherwise (all of the 32-bit mode)."""
@@ -948,10 +959,10 @@ def diff_attention(ctx, q, out, gate, cache, nh: int, nkv: int, kd: int, vd: int
         diff_attention_mma(q, out, gate, cache, b.seq_q_start_d, b.seq_q_len_d, b.seq_pos_start_d, b.n_seqs,
                            b.max_q_len, longest, any(short), not all(short), nh, nkv, kd, vd, window, scale, lam,
                            eps, out_scale, ctx.runtime.status,
-                           alloc=lambda n: ctx.ws.alloc((n,), torch.float32))
+                           alloc=lambda n: ctx.ws.alloc((n,), torch.float32), chunk=chunk)
     else:
         diff_attention_simt(q, out, gate, cache, b.positions, b.row_seq, nh, nkv, kd, vd, window, scale, lam, eps,
-                            out_scale, ctx.runtime.status)
+                            out_scale, ctx.runtime.status, chunk=chunk)
 
 
 _DIFF_MMA = [os.environ.get("FLAMBEAU_DIFF_ATTN_MMA", "1") != "0"]
@@ -971,14 +982,19 @@ QK_NORM_REACH = {None: 0, "none": 0, "head": 1, "projection": 2}
 
 def qk_norm_rope_kv_write(proj: torch.Tensor, q_weight, k_weight, reach, eps: float, weight_offset: float, cos, sin,
                           half: int, q_out: torch.Tensor, cache, positions, row_seq, nh: int, nkv: int, hd: int,
-                          vd: int, status, n_partials: int = 1, partial_stride: int = 0, v_off: int | None = None) -> None:
+                          vd: int, status, n_partials: int = 1, partial_stride: int = 0, v_off: int | None = None,
+                          bias=None, maps: int = 1) -> None:
     """proj: float32 rows [q: nh*hd | k: nkv*hd | v: nkv*vd] (possibly split-K shares; v_off: the column the values
     begin at where that is not right behind the keys; the keys' own first column: the values are the keys as projected).  q and k pass an RMS norm
     whose reach is a head ('head': weights [hd]) or the whole projection ('projection': weights [nh*hd] and
     [nkv*hd]) or none, then the rotation of the first 2*half dimensions of every head (cos/sin float32 [n, half]);
-    q goes to q_out in its dtype, k and v into the cache's pages when the view is writable."""
-    _cuda(proj, q_weight, k_weight, cos, sin, q_out, positions, row_seq, status)
+    q goes to q_out in its dtype, k and v into the cache's pages when the view is writable.  bias (optional, over the q,
+    k and v columns, contiguous) is added to the projection first.  maps: how many neighbouring heads of q and of k
+    belong to one head with several score maps: nh and nkv count the maps, the cache has nkv / maps key/value heads
+    whose key rows hold the maps side by side."""
+    _cuda(proj, q_weight, k_weight, cos, sin, q_out, positions, row_seq, status, bias)
     n = proj.shape[0]
+    nv = nkv // maps
     code = QK_NORM_REACH[reach]
     if proj.dtype != torch.float32 or tuple(q_out.shape) != (n, nh * hd):
         raise KernelError("qk_norm_rope_kv_write: float32 projection rows and q [n, heads * size] wanted")
@@ -989,15 +1005,18 @@ def qk_norm_rope_kv_write(proj: torch.Tensor, q_weight, k_weight, reach, eps: fl
             raise KernelError("qk_norm_rope_kv_write: the norm weights do not fit the norm's reach")
     k_pool, v_pool = cache.k_pool, cache.v_pool
     n_pages = k_pool.shape[0]
-    if tuple(k_pool.shape) != (n_pages, nkv, cache.page_size, hd) or tuple(v_pool.shape) != (n_pages, nkv, cache.page_size, vd) \
+    if bias is not None and (bias.numel() < (nh + nkv) * hd + nv * vd or not bias.is_contiguous()
+                             or (code and bias.dtype != q_weight.dtype)):
+        raise KernelError("qk_norm_rope_kv_write: the bias covers the q, k and v columns in the norm weights' dtype")
+    if tuple(k_pool.shape) != (n_pages, nv, cache.page_size, maps * hd) or tuple(v_pool.shape) != (n_pages, nv, cache.page_size, vd) \
             or not k_pool.is_contiguous() or not v_pool.is_contiguous() or k_pool.dtype != q_out.dtype:
         raise KernelError("qk_norm_rope_kv_write: the cache pools do not fit the head sizes")
     check(lib().fb_qk_norm_rope_kv_write(
-        proj.data_ptr(), _rows(proj), int(n_partials), int(partial_stride), _ptr(q_weight), _ptr(k_weight),
-        dtype_code(q_weight) if q_weight is not None else 0, code, float(eps), float(weight_offset), _ptr(cos),
+        proj.data_ptr(), _rows(proj), int(n_partials), int(partial_stride), _ptr(bias), _ptr(q_weight), _ptr(k_weight),
+        dtype_code(q_weight if q_weight is not None else bias) if q_weight is not None or bias is not None else 0, code, float(eps), float(weight_offset), _ptr(cos),
         _ptr(sin), int(half), q_out.data_ptr(), _rows(q_out), dtype_code(q_out), positions.data_ptr(),
         row_seq.data_ptr(), cache.block_table.data_ptr(), cache.block_table.stride(0), _ptr(cache.table_base),
-        int(cache.table_head), k_pool.data_ptr(), v_pool.data_ptr(), cache.page_size, n_pages, n, nh, nkv, hd, vd,
+        int(cache.table_head), k_pool.data_ptr(), v_pool.data_ptr(), cache.page_size, n_pages, n, nh, nkv, int(maps), hd, vd,
         (nh + nkv) * hd if v_off is None else int(v_off),
         1 if cache.writable else 0, status.data_ptr(), _stream()), "qk_norm_rope_kv_write")
 
@@ -1007,26 +1026,29 @@ def qk_norm_rope_kv_write(proj: torch.Tensor, q_weight, k_weight, reach, eps: fl
 # ---------------------------------------------------------------------------
 def gdr_prepare(proj, conv_w, taps: int, a_log, dt_bias, state, tail_off: int, batch, qkv, beta, decay, G: int,
                 H: int, dk: int, dv: int, q_scale: float, unit_eps: float, n_partials: int = 1,
-                partial_stride: int = 0) -> None:
+                partial_stride: int = 0, b_off: int | None = None, a_off: int | None = None) -> None:
     """The step's tokens made ready for the recurrence (csrc/gated_delta.cu: gdr_prepare, gdr_conv_tail).  proj:
-    float32 rows [q | k | v | b | a | gate] (possibly shares); state: float32 [slots, floats per slot] with the
-    convolution's tail at `tail_off`; qkv, beta, decay: float32 outputs [n, C], [n, H], [n, H]."""
+    float32 rows [q | k | v | ...] (possibly shares), with what beta and the decay are made of in the columns from b_off
+    and a_off on (default: right behind v, b then a); state: float32 [slots, floats per slot] with the convolution's tail
+    at `tail_off`; qkv, beta, decay: float32 outputs [n, C], [n, H], [n, H].  decay (with a_log and dt_bias) None: no
+    decay per head is formed."""
     _cuda(proj, conv_w, a_log, dt_bias, state, qkv, beta, decay)
     n = proj.shape[0]
     C = 2 * G * dk + H * dv
     if proj.dtype != torch.float32 or state.dtype != torch.float32 or not state.is_contiguous() or state.dim() != 2 \
-            or tuple(qkv.shape) != (n, C) or tuple(beta.shape) != (n, H) or tuple(decay.shape) != (n, H) \
+            or tuple(qkv.shape) != (n, C) or tuple(beta.shape) != (n, H) \
+            or (decay is not None and (tuple(decay.shape) != (n, H) or not conv_w.dtype == a_log.dtype == dt_bias.dtype)) \
             or tuple(conv_w.shape) != (C, taps) or not conv_w.is_contiguous() \
-            or not (conv_w.dtype == a_log.dtype == dt_bias.dtype) \
-            or any(t.dtype != torch.float32 or not t.is_contiguous() for t in (qkv, beta, decay)):
+            or any(t is not None and (t.dtype != torch.float32 or not t.is_contiguous()) for t in (qkv, beta, decay)):
         raise KernelError("gated delta: bad shapes or dtypes")
     if state.shape[1] < tail_off + (taps - 1) * C:
         raise KernelError("gated delta: the state slot is too small for the convolution's tail")
     check(lib().fb_gdr_prepare(proj.data_ptr(), _rows(proj), int(n_partials), int(partial_stride), conv_w.data_ptr(),
-                               int(taps), a_log.data_ptr(), dt_bias.data_ptr(), dtype_code(conv_w), state.data_ptr(),
+                               int(taps), C if b_off is None else int(b_off), C + H if a_off is None else int(a_off),
+                               _ptr(a_log), _ptr(dt_bias), dtype_code(conv_w), state.data_ptr(),
                                state.stride(0), int(tail_off), batch.row_seq.data_ptr(), batch.seq_q_start_d.data_ptr(),
                                batch.seq_q_len_d.data_ptr(), batch.seq_slot_d.data_ptr(), batch.n_seqs,
-                               qkv.data_ptr(), beta.data_ptr(), decay.data_ptr(), n, G, H, dk, dv, float(q_scale),
+                               qkv.data_ptr(), beta.data_ptr(), _ptr(decay), n, G, H, dk, dv, float(q_scale),
                                float(unit_eps), _stream()), "gdr_prepare")
 
 
@@ -1042,15 +1064,77 @@ def gdr_recurrent(qkv, beta, decay, state, batch, o, G: int, H: int, dk: int, dv
           "gdr_recurrent")
 
 
+def gdr_channel_recurrent(qkv, beta, decay, state, batch, o, G: int, H: int, dk: int, dv: int) -> None:
+    """S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q over the step's tokens of every request, with one
+    decay per head and key channel (decay float32 [n, H * dk]); the state as in gdr_recurrent."""
+    _cuda(qkv, beta, decay, state, o)
+    n = qkv.shape[0]
+    if o.dtype != torch.float32 or not o.is_contiguous() or o.shape[1] != H * dv or state.shape[1] < H * dk * dv \
+            or decay.dtype != torch.float32 or tuple(decay.shape) != (n, H * dk) or not decay.is_contiguous() \
+            or tuple(qkv.shape) != (n, 2 * G * dk + H * dv) or state.dtype != torch.float32 or not state.is_contiguous():
+        raise KernelError("gated delta: bad output, decay or state")
+    check(lib().fb_gdr_channel_recurrent(qkv.data_ptr(), beta.data_ptr(), decay.data_ptr(), state.data_ptr(),
+                                         state.stride(0), batch.seq_q_start_d.data_ptr(), batch.seq_q_len_d.data_ptr(),
+                                         batch.seq_slot_d.data_ptr(), batch.n_seqs, o.data_ptr(), G, H, dk, dv, _stream()),
+          "gdr_channel_recurrent")
+
+
+LOW_RANK_FUNCTIONS = {"plain": 0, "sigmoid": 1, "decay": 2}
+
+
+@dataclass(frozen=True)
+class LowRankMap:
+    """y = f(w z + bias) with z the `mid_off`-th and following columns of a projection: w [N, R], out float32 [n, N].
+    function 'plain', 'sigmoid', or 'decay': exp(-exp(log_rate[c // group]) * softplus(.))."""
+    w: torch.Tensor
+    mid_off: int
+    out: torch.Tensor
+    function: str = "plain"
+    bias: torch.Tensor | None = None
+    log_rate: torch.Tensor | None = None
+    group: int = 1
+
+
+def low_rank_maps(proj: torch.Tensor, maps, n_partials: int = 1, partial_stride: int = 0) -> None:
+    """One or two LowRankMaps of the same projection rows (float32, possibly shares) in one launch
+    (csrc/low_rank.cu)."""
+    n = proj.shape[0]
+    if proj.dtype != torch.float32 or not 1 <= len(maps) <= 2:
+        raise KernelError("low_rank_maps: float32 projection rows and one or two maps wanted")
+    _cuda(proj)
+    for m in maps:
+        _cuda(m.w, m.out, m.bias, m.log_rate)
+        N, R = m.w.shape
+        if m.w.dtype != maps[0].w.dtype or not m.w.is_contiguous() or m.out.dtype != torch.float32 \
+                or tuple(m.out.shape) != (n, N) or not m.out.is_contiguous() or proj.shape[1] < m.mid_off + R \
+                or any(t is not None and (t.dtype != m.w.dtype or not t.is_contiguous()) for t in (m.bias, m.log_rate)) \
+                or (m.bias is not None and m.bias.numel() != N) \
+                or (m.function == "decay" and (m.log_rate is None or m.log_rate.numel() * m.group < N)):
+            raise KernelError("low_rank_maps: shapes or dtypes do not agree")
+    k = len(maps)
+    ptrs, ints = ctypes.c_void_p * k, ctypes.c_int * k
+    check(lib().fb_low_rank_maps(
+        proj.data_ptr(), _rows(proj), int(n_partials), int(partial_stride), n, k, ptrs(*[m.w.data_ptr() for m in maps]),
+        dtype_code(maps[0].w), ints(*[int(m.mid_off) for m in maps]), ints(*[m.w.shape[1] for m in maps]),
+        ints(*[m.w.shape[0] for m in maps]), ints(*[LOW_RANK_FUNCTIONS[m.function] for m in maps]),
+        ptrs(*[_ptr(m.bias) or None for m in maps]), ptrs(*[_ptr(m.log_rate) or None for m in maps]),
+        ints(*[int(m.group) for m in maps]), ptrs(*[m.out.data_ptr() for m in maps]), _stream()), "low_rank_maps",
+        (n, sum(m.w.shape[0] for m in maps), maps[0].w.shape[1]))
+
+
+GDR_GATES = {"silu": 0, "sigmoid": 1, None: 2}
+
+
 def gdr_out_norm(o, proj, gate_off: int, weight, eps: float, out, H: int, dv: int, n_partials: int = 1,
-                 partial_stride: int = 0) -> None:
-    """out = o / rms(o) * weight * silu(gate) per head, the gate taken from the projection rows at `gate_off`."""
+                 partial_stride: int = 0, gate: str | None = "silu") -> None:
+    """out = o / rms(o) * weight * act(gate) per head, the gate taken from the projection rows at `gate_off`; `gate` names
+    act (GDR_GATES; None: the gate as it is)."""
     _cuda(o, proj, weight, out)
     n = o.shape[0]
     if tuple(out.shape) != (n, H * dv) or not out.is_contiguous() or weight.numel() != dv:
         raise KernelError("gated delta: bad output")
     check(lib().fb_gdr_out_norm(o.data_ptr(), proj.data_ptr(), _rows(proj), int(n_partials), int(partial_stride),
-                                int(gate_off), weight.data_ptr(), dtype_code(weight), float(eps), out.data_ptr(),
+                                int(gate_off), GDR_GATES[gate], weight.data_ptr(), dtype_code(weight), float(eps), out.data_ptr(),
                                 dtype_code(out), n, H, dv, _stream()), "gdr_out_norm")
 
 
@@ -1130,10 +1214,11 @@ def moe_combine(expert_out, pair_place, share, shared_out, shared_partials: int,
 # a norm that centres; a weighted mean over depth; a convolution over time in front of a sublayer
 # ---------------------------------------------------------------------------
 def add_layer_norm(x: torch.Tensor, delta, weight: torch.Tensor, eps: float, out: torch.Tensor, rows=None,
-                   n_partials: int = 1, n_rows: int | None = None, partial_stride: int = 0) -> None:
-    """out[j] = (v - mean v) / sqrt(var v + eps) * weight with v = x[r] + sum_p delta_p[r], r = rows[j] or j; without
-    `rows` the sum is also written back to x.  delta: float32 [n, H] or the first of n_partials slabs."""
-    _cuda(x, delta, weight, out, rows)
+                   n_partials: int = 1, n_rows: int | None = None, partial_stride: int = 0, delta_bias=None) -> None:
+    """out[j] = (v - mean v) / sqrt(var v + eps) * weight with v = x[r] + sum_p delta_p[r] + delta_bias, r = rows[j] or j;
+    without `rows` the sum is also written back to x.  delta: float32 [n, H] or the first of n_partials slabs (or None);
+    delta_bias: a vector [H] in the weight's dtype (or None)."""
+    _cuda(x, delta, weight, out, rows, delta_bias)
     _i32(rows, "rows")
     H = x.shape[1]
     n_out = rows.numel() if rows is not None else (x.shape[0] if n_rows is None else n_rows)
@@ -1148,8 +1233,11 @@ def add_layer_norm(x: torch.Tensor, delta, weight: torch.Tensor, eps: float, out
             stride = int(partial_stride)
             if stride <= 0:
                 raise KernelError("add_layer_norm: several slabs need their stride")
+    if delta_bias is not None and (delta_bias.numel() != H or delta_bias.dtype != weight.dtype
+                                   or not delta_bias.is_contiguous()):
+        raise KernelError("add_layer_norm: the bias is a contiguous vector of the stream's width in the weight's dtype")
     check(lib().fb_add_layernorm(x.data_ptr(), _ptr(delta), int(n_partials) if delta is not None else 0, stride,
-                                 weight.data_ptr(), dtype_code(weight), out.data_ptr(), dtype_code(out), _ptr(rows),
+                                 _ptr(delta_bias), weight.data_ptr(), dtype_code(weight), out.data_ptr(), dtype_code(out), _ptr(rows),
                                  n_out, H, float(eps), _stream()), "add_layer_norm")
 
 
@@ -1235,22 +1323,26 @@ def mla_latents(proj, Rq: int, wq, cq, kv_off: int, Rc: int, r: int, wkv, eps: f
                 positions, row_seq, status, n_partials: int = 1, partial_stride: int = 0,
                 pairing: str = "neighbours") -> None:
     """cq = rmsnorm(proj[:, :Rq]) * wq; with a writable cache also the token's cache row [rmsnorm(proj[:, kv_off:
-    kv_off + Rc]) * wkv | rot(proj[:, kv_off + Rc : kv_off + Rc + r])] (csrc/latent_attention.cu)."""
+    kv_off + Rc]) * wkv | rot(proj[:, kv_off + Rc : kv_off + Rc + r])] (csrc/latent_attention.cu).  Rq = 0 (wq and cq
+    None): only the cache row."""
     _cuda(proj, wq, cq, wkv, cos, sin, positions, row_seq, status)
     n = proj.shape[0]
-    if proj.dtype != torch.float32 or wq.numel() != Rq or tuple(cq.shape) != (n, Rq) or not cq.is_contiguous():
+    if proj.dtype != torch.float32 or (Rq > 0 and (wq.numel() != Rq or tuple(cq.shape) != (n, Rq) or not cq.is_contiguous())):
         raise KernelError("latent attention: bad shapes")
     pool = cache.k_pool if cache is not None and cache.writable else None
+    if Rq == 0 and pool is None:
+        raise KernelError("latent attention: neither a query's latent nor a cache row to form")
+    weight, row_dtype = (wq, cq) if Rq > 0 else (wkv, pool)
     if pool is not None:
-        if tuple(pool.shape[1:]) != (1, cache.page_size, Rc + r) or not pool.is_contiguous() or pool.dtype != cq.dtype \
-                or wkv.numel() != Rc or wkv.dtype != wq.dtype or proj.shape[1] < kv_off + Rc + r:
+        if tuple(pool.shape[1:]) != (1, cache.page_size, Rc + r) or not pool.is_contiguous() or pool.dtype != row_dtype.dtype \
+                or wkv.numel() != Rc or wkv.dtype != weight.dtype or proj.shape[1] < kv_off + Rc + r:
             raise KernelError("latent attention: the cache rows do not fit the latent")
     check(lib().fb_mla_latents(
-        proj.data_ptr(), _rows(proj), int(n_partials), int(partial_stride), Rq, wq.data_ptr(), cq.data_ptr(), kv_off,
-        Rc, r, _ptr(wkv), dtype_code(wq), float(eps), _ptr(cos), _ptr(sin), half, ROTARY_PAIRING[pairing],
+        proj.data_ptr(), _rows(proj), int(n_partials), int(partial_stride), Rq, _ptr(wq), _ptr(cq), kv_off,
+        Rc, r, _ptr(wkv), dtype_code(weight), float(eps), _ptr(cos), _ptr(sin), half, ROTARY_PAIRING[pairing],
         _ptr(positions), _ptr(row_seq),
         _ptr(cache.block_table) if pool is not None else 0, cache.block_table.stride(0) if pool is not None else 0,
-        _ptr(cache.table_base) if pool is not None else 0, _ptr(pool), dtype_code(cq),
+        _ptr(cache.table_base) if pool is not None else 0, _ptr(pool), dtype_code(row_dtype),
         cache.page_size if pool is not None else 1, pool.shape[0] if pool is not None else 0, n, status.data_ptr(),
         _stream()), "mla_latents")
 

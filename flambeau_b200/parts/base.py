@@ -49,6 +49,7 @@ class KVRequirement:
     v_head_dim: int = 0      # elements of a value row where it differs from a key row (0: the same)
     values_in_keys: bool = False   # the key rows are the values as well: one pool serves as both, nothing is kept twice
     keep_first: int = 0      # under a window: the first keys of a request stay visible to every later query
+    chunk: int = 0           # C > 0 = a query sees the keys of its own chunk of C positions (counted from position 0)
 
     @property
     def value_dim(self) -> int:
@@ -56,8 +57,9 @@ class KVRequirement:
 
     @property
     def release_window(self) -> int:
-        """The window by which the cache manager gives pages back (0: never before the request ends)."""
-        return self.window
+        """How many keys up to a query's own stay live at most under the rules by which the cache manager gives pages
+        back (0: no page is given back before the request ends)."""
+        return min((n for n in (self.window, self.chunk) if n > 0), default=0)
 
     def kept_pages(self, page_size: int) -> int:
         """Pages at a request's start that a window never gives back: those that hold its kept first keys."""

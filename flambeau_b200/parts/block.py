@@ -95,15 +95,19 @@ class PreNormBlock(Part):
         return self._state
 
     def _normed_input(self, ctx, norm, input_map, offset, stream, call, h):
-        """h = input_map(norm(x + pending)) (or the norm alone), the pending output added to the stream on the way."""
+        """h = input_map(norm(x + pending)) (or the norm alone), the pending output added to the stream on the way (and the
+        bias that a part has left to this norm: ctx.pending_bias)."""
+        extra = {}
+        if ctx.pending_bias is not None:
+            extra["delta_bias"], ctx.pending_bias = ctx.pending_bias, None
         if input_map is None:
             norm.add_norm(ctx, stream.x, stream.pending, h, n_partials=stream.pending_slabs,
-                          delta_norm=stream.pending_norm)
+                          delta_norm=stream.pending_norm, **extra)
             return
         with ctx.ws.scope():
             rows = ctx.ws.alloc((ctx.n_tokens, stream.x.shape[1]), torch.float32)
             norm.add_norm(ctx, stream.x, stream.pending, rows, n_partials=stream.pending_slabs,
-                          delta_norm=stream.pending_norm)
+                          delta_norm=stream.pending_norm, **extra)
             state = ctx.cache(call).state
             input_map.forward(ctx, rows, h, state.view(state.shape[0], -1) if state is not None else None, offset)
 
@@ -113,7 +117,10 @@ class PreNormBlock(Part):
         self._normed_input(ctx, self.mixer_norm, self.mixer_input, self._offsets[0], stream, call, h)
         stream.pending_norm = None
         ctx.pending_slabs = 1                 # a part that leaves split-K shares in ctx.delta_slabs says how many
+        # the mixer's output bias joins the stream in the norm ahead of the feed-forward, where there is one that takes it
+        ctx.bias_can_wait = getattr(self.feed_forward_norm, "takes_bias", False)
         self.mixer.forward(ctx, h, delta, call)
+        ctx.bias_can_wait = False
         stream.pending, stream.pending_slabs = delta, ctx.pending_slabs
         if self.feed_forward is not None:
             self._normed_input(ctx, self.feed_forward_norm, self.feed_forward_input, self._offsets[1], stream, call, h)

@@ -58,13 +58,16 @@ class TokenEmbedding(Part):
 class LMHead(Part):
     """logits = h W^T (times `scale`) in float32, for the wanted rows only; a tied head reuses
     the embedding table (crates/forward/src/core/composites/output_head.rs:90-132;
-    crates/models/qwen35-v2/src/loader.rs:219-223)."""
+    crates/models/qwen35-v2/src/loader.rs:219-223).  `softcap` (> 0): every logit passes cap * tanh(logit / cap)."""
     graph_safe = True
     category = "head"
 
     def __init__(self, runtime=None, prefix="", *, vocab: int, width: int, tied_to: str | None = None,
-                 init_std: float = 0.02, weight_name: str = "weight", scale: float = 1.0):
+                 init_std: float = 0.02, weight_name: str = "weight", scale: float = 1.0, softcap: float = 0.0):
         super().__init__(runtime, prefix)
+        self.softcap = float(softcap or 0.0)
+        if self.softcap < 0.0:
+            raise ValueError(f"output head: softcap = {softcap} must be positive (0 or None: none)")
         self.vocab, self.width, self.tied_to, self.init_std = int(vocab), int(width), tied_to, init_std
         self.weight_name, self.scale = weight_name, float(scale)
         self.proj = None
@@ -83,6 +86,8 @@ class LMHead(Part):
         self.proj(ctx, h_rows, logits)
         if self.scale != 1.0:
             logits.mul_(self.scale)          # float32, the wanted rows only
+        if self.softcap:
+            ops.softcap_rows(logits, self.softcap)
 
 
 register_part("embedding", "token_embedding", TokenEmbedding)

@@ -86,7 +86,7 @@ class GatedMLP(FeedForward):
 
 class PlainMLP(FeedForward):
     """d = act(h Wu^T) Wd^T: no gate, no bias, no routing.  `activation` names one of the kernels' plain activations
-    (kernels.ops.PLAIN_ACTIVATIONS: relu_squared, silu, gelu_tanh).  Over a prompt's portion the activation runs in
+    (kernels.ops.PLAIN_ACTIVATIONS: relu_squared, silu, gelu, gelu_tanh).  Over a prompt's portion the activation runs in
     the first product's epilogue; with few rows the product leaves float32 split-K shares and the activation kernel
     adds them.  `names`: what the up and down tensors are called behind the prefix."""
     graph_safe = True

@@ -57,6 +57,7 @@ class LayerNorm(Norm):
     a weight and no bias.  Mean, variance (from the deviations) and the product are float32; the stream stays
     float32.  The tensor is `<prefix><weight_name>`."""
     graph_safe = True
+    takes_bias = True                 # add_norm(delta_bias=...): a vector that joins the stream with the delta
 
     def __init__(self, runtime=None, prefix="", *, width: int, eps: float, init=("one_plus_normal", 0.02),
                  weight_name: str = "weight"):
@@ -73,14 +74,14 @@ class LayerNorm(Norm):
     def own_weights(self):
         return [self.weight]
 
-    def add_norm(self, ctx, x, delta, out, rows=None, n_partials: int = 1, delta_norm=None):
+    def add_norm(self, ctx, x, delta, out, rows=None, n_partials: int = 1, delta_norm=None, delta_bias=None):
         if delta_norm is not None:
             raise ValueError("the centring norm adds a part's output as it is; a norm behind the part is not fused here")
         if n_partials == 0 or delta is None:     # the stream already holds the sum
             delta = None
         stride = ctx.delta_slabs.stride(0) if n_partials > 1 else 0
         ops.add_layer_norm(x, delta, self.weight, self.eps, out, rows=rows, n_partials=n_partials,
-                           n_rows=ctx.n_tokens, partial_stride=stride)
+                           n_rows=ctx.n_tokens, partial_stride=stride, delta_bias=delta_bias)
 
     def normalize(self, ctx, x, out):
         ops.add_layer_norm(x, None, self.weight, self.eps, out, n_rows=x.shape[0])

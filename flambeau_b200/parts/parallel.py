@@ -59,8 +59,8 @@ class ParallelMixers(Mixer):
     def forward(self, ctx, h, out, call):
         n = ctx.n_tokens
         # a branch's output has to pass its norm before it may join the stream: no product adds to the stream here
-        kept = (ctx.stream_x, ctx.delta_slabs, ctx.delta)
-        ctx.stream_x = None
+        kept = (ctx.stream_x, ctx.delta_slabs, ctx.delta, ctx.bias_can_wait)
+        ctx.stream_x, ctx.bias_can_wait = None, False
         try:
             with ctx.ws.scope():
                 mix = []
@@ -72,7 +72,7 @@ class ParallelMixers(Mixer):
                     mix.append((y[0], max(1, ctx.pending_slabs), y.stride(0), weight, coef))
                 ops.branch_norm_mix(mix, self.eps, out, n)
         finally:
-            ctx.stream_x, ctx.delta_slabs, ctx.delta = kept
+            ctx.stream_x, ctx.delta_slabs, ctx.delta, ctx.bias_can_wait = kept
         ctx.pending_slabs = 1
 
 

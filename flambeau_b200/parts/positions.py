@@ -13,7 +13,13 @@ from .spec import register_part
 def rotary_frequencies(theta: float, rotary_dim: int, stretch: dict | None = None) -> tuple:
     """(frequencies of the rotary_dim / 2 pairs, factor on cos and sin), formed in float64: f_i = theta^(-2i/rot).
 
-    `stretch` (optional: factor, original, fast, slow) lengthens the slow waves so that positions beyond `original`
+    `stretch` (optional) comes in two rules, told apart by their constants.
+
+    factor, original, low, high: with the wave length l = 2 pi / f, waves shorter than original / high keep their
+    frequency, those longer than original / low get f / factor, and between the two, with s = (original / l - low) /
+    (high - low), the frequency is (1 - s) f / factor + s f.  cos and sin are as they are.
+
+    factor, original, fast, slow: lengthens the slow waves so that positions beyond `original`
     stay within the angles seen in training: with index(t) = rot * ln(original / (2 pi t)) / (2 ln theta) the pair
     index whose wave makes t turns over `original` positions, lo = max(floor(index(fast)), 0),
     hi = min(ceil(index(slow)), rot - 1) and ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), the frequency of
@@ -24,6 +30,18 @@ def rotary_frequencies(theta: float, rotary_dim: int, stretch: dict | None = Non
     if not stretch:
         return freqs, 1.0
     factor, original = float(stretch["factor"]), float(stretch["original"])
+    if "low" in stretch:
+        low, high = float(stretch["low"]), float(stretch["high"])
+
+        def banded(f):
+            turns = original * f / (2.0 * math.pi)           # original / wave length
+            if turns >= high:
+                return f
+            if turns <= low:
+                return f / factor
+            s = (turns - low) / (high - low)
+            return (1.0 - s) * f / factor + s * f
+        return [banded(f) for f in freqs], 1.0
 
     def index(turns):
         return rotary_dim * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(theta))
