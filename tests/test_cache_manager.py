@@ -380,3 +380,46 @@ def test_snapshot_and_restore_keep_the_kept_pages():
     assert all(p >= 0 for p in list(cm.requests["b"].pages[0])[:2]), "the kept pages are still there"
     cm.release_all()
     assert cm.free_pages() == [20]
+
+
+@pytest.mark.parametrize("chunk", [1, 5, 8, 20, 24, 64])
+def test_a_chunk_is_given_back_when_the_request_leaves_it(chunk):
+    """A query sees its own chunk of positions only: once the next position lies in another chunk, the pages wholly below
+    that chunk's start are dead, whatever the portions were; a long request runs in a pool of a few pages."""
+    page = 8
+    req = KVRequirement(1, 8, 0, chunk=chunk)
+    assert req.release_window == chunk and KVRequirement(1, 8, 24, chunk=chunk).release_window == min(24, chunk)
+    cm = CacheManager([CallPlan(kv=req), CallPlan(kv=KVRequirement(1, 8, 0))], max_tokens=640, page_size=page, max_requests=2,
+                      device="cpu", dtype=torch.float32, max_seq_len=600, max_step_tokens=16)
+    assert cm.n_groups == 2, "chunked layers have pages of their own"
+    cm.admit("a")
+    length = 0
+    for k in [1, 2, 16, 3, 9, 16, 16, 1, 1, 7, 16, 16, 13, 2, 5, 16, 16, 16] * 2:
+        cm.reserve("a", k)
+        live = [p for p in cm.requests["a"].pages[0] if p >= 0]
+        assert len(live) <= -(-(chunk + 16) // page) + 2
+        cm.commit("a", k)
+        length += k
+        first = length // chunk * chunk
+        for j, p in enumerate(cm.requests["a"].pages[0]):
+            assert (p < 0) == ((j + 1) * page <= first), (length, j)
+        assert all(p >= 0 for p in cm.requests["a"].pages[1]), "the other group keeps everything"
+        cm.check_invariants()
+    snap = cm.snapshot("a")
+    cm.release("a")
+    cm.restore("b", snap)
+    assert cm.length("b") == length and cm.first_live_page("b", 0) == length // chunk * chunk // page
+    cm.check_invariants()
+    cm.release_all()
+    assert cm.free_pages() == [80, 80]
+
+
+def test_a_reader_of_a_chunked_cache_has_its_chunks():
+    def build(owner, reader):
+        return CacheManager([CallPlan(kv=owner), CallPlan(kv=reader, cache_from=0)], max_tokens=64, page_size=16,
+                            max_requests=1, device="cpu", dtype=torch.float32)
+    for reader in (KVRequirement(2, 16, 0), KVRequirement(2, 16, 8), KVRequirement(2, 16, 0, chunk=16)):
+        with pytest.raises(ValueError, match="chunks"):
+            build(KVRequirement(2, 16, 0, chunk=32), reader)
+    build(KVRequirement(2, 16, 0, chunk=32), KVRequirement(2, 16, 0, chunk=32))
+    build(KVRequirement(2, 16, 0), KVRequirement(2, 16, 0, chunk=32))
