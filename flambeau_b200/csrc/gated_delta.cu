@@ -102,6 +102,108 @@ gdr_prepare_kernel(const float* __restrict__ proj, long proj_stride, int n_parti
     }
 }
 
+// The same for up to four taps and heads of up to 256 whose sizes are multiples of 4: a warp takes a head of ROWS
+// neighbouring rows, four neighbouring channels a lane (16-byte loads and stores, NV groups of them), and the rows' inputs
+// form a window in registers, so that a row's input is fetched once and not once a tap.
+template <typename TW, int TAPS, int NV, int ROWS>
+__global__ void __launch_bounds__(128)
+gdr_prepare_vec_kernel(const float* __restrict__ proj, long proj_stride, int n_partials, long partial_stride,
+                       const TW* __restrict__ conv_w, int b_off, int a_off, const TW* __restrict__ a_log,
+                       const TW* __restrict__ dt_bias, const float* __restrict__ state, long state_stride, long tail_off,
+                       const int* __restrict__ row_seq, const int* __restrict__ seq_q_start, const int* __restrict__ seq_slot,
+                       float* __restrict__ qkv, float* __restrict__ beta, float* __restrict__ decay, int n, int G, int H,
+                       int dk, int dv, float q_scale, float unit_eps) {
+    fb_pdl_launch_dependents();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int units = 2 * G + H, qk = G * dk, C = 2 * qk + H * dv;
+    const long item = (long)blockIdx.x * 4 + warp;
+    const int unit = (int)(item % units), row0 = (int)(item / units) * ROWS;
+    if (row0 >= n) return;
+    const bool is_v = unit >= 2 * G;
+    const int width = is_v ? dv : dk;
+    const int base = is_v ? 2 * qk + (unit - 2 * G) * dv : unit * dk;    // q heads, then k heads, then v heads
+    float w[NV][4 * TAPS];                             // [channel][tap]
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int d = 4 * lane + 128 * i;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) {
+            const float4 v = d < width ? Vec4<TW>::load(conv_w + (size_t)(base + d) * TAPS + 4 * j) : make_float4(0.f, 0.f, 0.f, 0.f);
+            w[i][4 * j] = v.x; w[i][4 * j + 1] = v.y; w[i][4 * j + 2] = v.z; w[i][4 * j + 3] = v.w;
+        }
+    }
+    fb_pdl_wait();
+    int place[ROWS];                                   // the rows' places within their requests' portions
+    const float* tail[ROWS];
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) {
+        const int seq = row_seq[min(row0 + r, n - 1)];
+        place[r] = row0 + r - seq_q_start[seq];
+        tail[r] = state + (size_t)seq_slot[seq] * state_stride + tail_off;
+    }
+    float y[NV][ROWS][4], sq[ROWS];
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) sq[r] = 0.0f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int d = 4 * lane + 128 * i;
+        const bool in = d < width;
+        float4 x[ROWS + TAPS - 1];                     // x[m]: the input of row row0 + m - (TAPS - 1)
+#pragma unroll
+        for (int m = 0; m < ROWS + TAPS - 1; ++m) {
+            const int off = m - (TAPS - 1);
+            // (a row ahead of row0 is wanted where it belongs to row0's portion)
+            const bool wanted = in && row0 + off < n && (off >= 0 || place[0] >= -off);
+            x[m] = wanted ? slab_sum4(proj + (size_t)(row0 + off) * proj_stride + base + d, n_partials, partial_stride)
+                          : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) {
+            float acc[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) {
+                const int back = TAPS - 1 - j;
+                float4 v = x[r + j];
+                if (place[r] < back)                   // before the portion: the kept inputs
+                    v = in ? Vec4<float>::load(tail[r] + (size_t)(TAPS - 1 + place[r] - back) * C + base + d)
+                           : make_float4(0.f, 0.f, 0.f, 0.f);
+                acc[0] = fmaf(w[i][j], v.x, acc[0]);
+                acc[1] = fmaf(w[i][TAPS + j], v.y, acc[1]);
+                acc[2] = fmaf(w[i][2 * TAPS + j], v.z, acc[2]);
+                acc[3] = fmaf(w[i][3 * TAPS + j], v.w, acc[3]);
+            }
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                y[i][r][u] = gdr_silu(acc[u]);
+                sq[r] = fmaf(y[i][r][u], y[i][r][u], sq[r]);
+            }
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) {
+        const int row = row0 + r;
+        float f = 1.0f;
+        if (!is_v) f = (unit < G ? q_scale : 1.0f) / sqrtf(fb_warp_sum(sq[r]) + unit_eps);    // (warp-uniform)
+        if (row >= n) break;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int d = 4 * lane + 128 * i;
+            if (d < width)
+                Vec4<float>::store(qkv + (size_t)row * C + base + d,
+                                   make_float4(y[i][r][0] * f, y[i][r][1] * f, y[i][r][2] * f, y[i][r][3] * f));
+        }
+        if (is_v && lane == 0) {
+            const int h = unit - 2 * G;
+            const float* pr = proj + (size_t)row * proj_stride;
+            beta[(size_t)row * H + h] = 1.0f / (1.0f + expf(-fb_slab_sum(pr, b_off + h, n_partials, partial_stride)));
+            if (decay) {
+                const float a = fb_slab_sum(pr, a_off + h, n_partials, partial_stride);
+                decay[(size_t)row * H + h] = expf(-expf(fb_to_float(a_log[h])) * gdr_softplus(a + fb_to_float(dt_bias[h])));
+            }
+        }
+    }
+}
+
 __global__ void gdr_conv_tail_kernel(const float* __restrict__ proj, long proj_stride, int n_partials, long partial_stride,
                                      int taps, float* __restrict__ state, long state_stride, long tail_off,
                                      const int* __restrict__ seq_q_start, const int* __restrict__ seq_q_len,
@@ -565,6 +667,30 @@ FB_API int fb_gdr_prepare(const float* proj, long long proj_stride, int n_partia
     if (n_partials < 1) n_partials = 1;
     FB_REQUIRE(dk <= 1024 && dv <= 1024, "gated delta: head sizes up to 1024 (key %d, value %d)", dk, dv);
     FB_REQUIRE(2 * G + H <= 65535, "gated delta: too many heads");
+    const size_t wsize = w_dtype == FB_BF16 ? 2 : 4;
+    const int widest = dk > dv ? dk : dv;
+    auto aligned = [](const void* p, size_t to) { return (uintptr_t)p % to == 0; };
+    const bool vec = taps <= 4 && dk % 4 == 0 && dv % 4 == 0 && widest <= 256 && proj_stride % 4 == 0 && partial_stride % 4 == 0 &&
+                     state_stride % 4 == 0 && tail_off % 4 == 0 && aligned(proj, 16) && aligned(state, 16) && aligned(qkv, 16) &&
+                     aligned(conv_w, 4 * wsize);
+    if (vec) {
+        // (a few rows: one a warp, so that the heads spread over the device; a portion: four)
+#define FB_GDP_LAUNCH(TAPS_, NV_, ROWS_)                                                                                     \
+        FB_DISPATCH_DTYPE(w_dtype, TW,                                                                                       \
+            (fb_launch((gdr_prepare_vec_kernel<TW, TAPS_, NV_, ROWS_>),                                                      \
+                       dim3((unsigned)(((long)((n + ROWS_ - 1) / ROWS_) * (2 * G + H) + 3) / 4)), dim3(128), 0, stream, proj, \
+                       (long)proj_stride, n_partials, (long)partial_stride, (const TW*)conv_w, b_off, a_off, (const TW*)a_log, \
+                       (const TW*)dt_bias, (const float*)state, (long)state_stride, (long)tail_off, row_seq, seq_q_start,     \
+                       seq_slot, qkv, beta, decay, n, G, H, dk, dv, q_scale, unit_eps)))
+#define FB_GDP_TAPS(TAPS_)                                                                                                   \
+        case TAPS_:                                                                                                          \
+            if (widest <= 128) { if (n <= 64) FB_GDP_LAUNCH(TAPS_, 1, 1); else FB_GDP_LAUNCH(TAPS_, 1, 4); }                   \
+            else { if (n <= 64) FB_GDP_LAUNCH(TAPS_, 2, 1); else FB_GDP_LAUNCH(TAPS_, 2, 4); }                                \
+            break;
+        switch (taps) { FB_GDP_TAPS(1) FB_GDP_TAPS(2) FB_GDP_TAPS(3) FB_GDP_TAPS(4) }
+#undef FB_GDP_TAPS
+#undef FB_GDP_LAUNCH
+    } else
     FB_DISPATCH_DTYPE(w_dtype, TW, {
         auto kernel = gdr_prepare_kernel<TW>;
         fb_launch(kernel, dim3(n, 2 * G + H), dim3(128), 0, stream, proj, (long)proj_stride, n_partials, (long)partial_stride,

@@ -590,6 +590,9 @@ FB_API int fb_gemm_tc_act(const void* X, long long lda, const void* W, long long
     FB_REQUIRE(((uintptr_t)X & 15) == 0 && ((uintptr_t)W & 15) == 0, "gemm_tc_act: operands must be 16-byte aligned");
     if (M == 0) return 0;
     const int BN = M <= 16 ? 16 : M <= 32 ? 32 : M <= 64 ? 64 : M <= 128 ? 128 : 256;
+    if (BN == 256 && o_dtype == FB_BF16 && fb_gemm_pair_plan(M, N, K, 1))
+        return fb_launch_gemm_pair(X, (long)lda, W, (long)ldw, out, o_dtype, (long)ldo, 0, 1, M, N, K, FbGate{0, 0.0f, 0.0f}, 0,
+                                   status, stream, act);
     CUtensorMap mw, mx;
     int rc = fb_tensor_map_bf16(&mw, W, N, K, (long)ldw, BK, BM);
     if (rc) return rc;

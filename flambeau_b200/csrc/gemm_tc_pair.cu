@@ -110,12 +110,12 @@ __device__ __forceinline__ PairUnit pair_unit(int u, int tiles_m, int tiles, int
     return w;
 }
 
-template <typename TO>
+template <typename TO, bool ACT>     // ACT: the epilogue applies the plain activation `plain_act`
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(P_THREADS, 1)
 gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                     const __grid_constant__ CUtensorMap map_o, int boxed_out,
                     TO* __restrict__ out, long ldo, long slab_stride, int M, int N, int K, int tiles_m, int tiles,
-                    int splits, int n_units, FbGate gated, int accumulate, int* status) {
+                    int splits, int n_units, FbGate gated, int plain_act, int accumulate, int* status) {
     constexpr int S = P_STAGES;
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
@@ -273,6 +273,10 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
 #pragma unroll
                         for (int q = 0; q < 16; ++q) v[q] = 0.0f;
                     }
+                    if constexpr (ACT) {
+#pragma unroll
+                        for (int q = 0; q < 16; ++q) v[q] = fb_plain_act(plain_act, v[q]);
+                    }
                     if (boxed_out) {
                         if (leader) bulk_wait_read();           // the box sent from this buffer, the one before last, has left it
                         asm volatile("bar.sync %0, 128;" ::"r"(2 + half_id) : "memory");
@@ -338,9 +342,9 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
     }
 }
 
-template <typename TO>
+template <typename TO, bool ACT = false>
 int launch_pair(const void* X, long lda, const void* W, long ldw, void* out, long ldo, long slab_stride, int splits,
-                int M, int N, int K, FbGate gated, int accumulate, int* status, cudaStream_t stream) {
+                int M, int N, int K, FbGate gated, int accumulate, int* status, cudaStream_t stream, int plain_act = 0) {
     CUtensorMap mw, mx;
     int rc = fb_tensor_map_bf16(&mw, W, N, K, ldw, PBK, PBM);
     if (rc) return rc;
@@ -351,7 +355,7 @@ int launch_pair(const void* X, long lda, const void* W, long ldw, void* out, lon
     const int boxed = fb_tensor_map_out(&mo, out, (int)sizeof(TO), M, gated.act ? N / 2 : N, ldo, splits, slab_stride,
                                         gated.act ? PBM / 2 : PBM, P_OUT_TOKENS);
     if (boxed < 0) return boxed;
-    auto kern = gemm_tc_pair_kernel<TO>;
+    auto kern = gemm_tc_pair_kernel<TO, ACT>;
     static bool configured[FB_MAX_DEVICES] = {};
     if (fb_needs_setup(configured)) {
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, P_SMEM_BYTES);
@@ -366,7 +370,7 @@ int launch_pair(const void* X, long lda, const void* W, long ldw, void* out, lon
     const int pairs = (int)(n_units < pair_slots() ? n_units : pair_slots());
     fb_launch_class(FB_LAUNCH_GEMM_PAIR, (kern), 2 * pairs, P_THREADS, P_SMEM_BYTES, stream, mw, mx, mo,
                     boxed == 0 ? 1 : 0, (TO*)out, ldo, slab_stride, M, N, K, tiles_m, (int)tiles, splits, (int)n_units,
-                    gated, accumulate, status);
+                    gated, plain_act, accumulate, status);
     return fb_check_launch("gemm_tc_pair");
 }
 
@@ -406,7 +410,12 @@ int fb_gemm_pair_plan(int M, int N, int K, int max_slabs) {
 
 int fb_launch_gemm_pair(const void* X, long lda, const void* W, long ldw, void* out, int o_dtype, long ldo,
                         long slab_stride, int splits, int M, int N, int K, FbGate gated, int accumulate, int* status,
-                        cudaStream_t stream) {
+                        cudaStream_t stream, int plain_act) {
+    if (plain_act) {
+        if (splits != 1 || accumulate || gated.act || o_dtype != FB_BF16)
+            return fb_fail(-1, "gemm_tc_pair: a plain activation needs a whole product in bfloat16 of its own");
+        return launch_pair<__nv_bfloat16, true>(X, lda, W, ldw, out, ldo, 0, 1, M, N, K, gated, 0, status, stream, plain_act);
+    }
     if (splits < 1 || (splits > 1 && (slab_stride <= 0 || o_dtype != FB_F32 || gated.act)))
         return fb_fail(-1, "gemm_tc_pair: %d shares of K need float32 slabs", splits);
     if (accumulate && (o_dtype != FB_F32 || splits != 1 || gated.act))

@@ -9,7 +9,8 @@
 int fb_gemm_pair_plan(int M, int N, int K, int max_slabs);
 // out[M,N] (or act(g)*u of alternating features into [M,N/2] when `gated` names an activation) = X[M,K] * W[N,K]^T; with splits > 1
 // share s of K goes to out + s * slab_stride (float32) and the caller adds the slabs.  accumulate: the whole float32
-// product is added to what `out` holds instead of replacing it.
+// product is added to what `out` holds instead of replacing it.  plain_act (an FbPlainAct code): applied to every element of
+// a whole bfloat16 product.
 int fb_launch_gemm_pair(const void* X, long lda, const void* W, long ldw, void* out, int o_dtype, long ldo,
                         long slab_stride, int splits, int M, int N, int K, FbGate gated, int accumulate, int* status,
-                        cudaStream_t stream);
+                        cudaStream_t stream, int plain_act = 0);

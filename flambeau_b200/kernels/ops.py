@@ -1238,7 +1238,8 @@ def add_layer_norm(x: torch.Tensor, delta, weight: torch.Tensor, eps: float, out
         raise KernelError("add_layer_norm: the bias is a contiguous vector of the stream's width in the weight's dtype")
     check(lib().fb_add_layernorm(x.data_ptr(), _ptr(delta), int(n_partials) if delta is not None else 0, stride,
                                  _ptr(delta_bias), weight.data_ptr(), dtype_code(weight), out.data_ptr(), dtype_code(out), _ptr(rows),
-                                 n_out, H, float(eps), _stream()), "add_layer_norm")
+                                 n_out, H, float(eps), _stream()), "add_layer_norm",
+          (n_out, H, min(int(n_partials), 1) if delta is not None else 0, 1 if delta_bias is not None else 0, 1 if rows is None else 0))
 
 
 def depth_average(x: torch.Tensor, delta, n_partials: int, partial_stride: int, history: torch.Tensor, count: int,

@@ -90,7 +90,7 @@ def main(argv=None) -> int:
     ap.add_argument("--prefill-tokens", type=int, default=2048)
     ap.add_argument("--skip-points", action="store_true", help="do not measure batch 1 and 64")
     ap.add_argument("--only", choices=["all", "headline", "mixed", "shapes", "timeline", "mma-issue", "zedivik", "nodepel", "fegizen", "tubepel",
-                                      "saropel"],
+                                      "saropel", "sisadra"],
                     default="all",
                     help="headline: the shape's own line only; mixed / shapes: that part only; timeline: the kernels "
                          "of one decode step at --batch as the device ran them (a table on stderr, 4 layers unless "
@@ -231,6 +231,18 @@ def main(argv=None) -> int:
             result = compare_saropel.run(sizes, args.layers or 4, args.batch, args.prefill_tokens, min(args.steps, 64),
                                          args.warmup, pk, gen, say)
         print(json.dumps({"impl": "ours", "metric": "Saropel beside Tubepel at equal size: decode and prefill tok/s, "
+                          "per-kernel microseconds per launch", "dtype": "bf16", "data": "synthetic", "peak": tag,
+                          "peaks": {"hbm_gbs": pk["hbm_gbs"], "bf16_tflops": pk["bf16_tflops"]},
+                          "compare": result, "clocks": clocks.summary()}))
+        return 0
+    if args.only == "sisadra":
+        from flambeau_b200.measure import compare_sisadra
+        with ClockSampler(0) as clocks:
+            time.sleep(0.3)
+            sizes = [k for k in args.sizes.split(",") if k in compare_sisadra.SIZES]
+            result = compare_sisadra.run(sizes, args.layers or 4, args.batch, args.prefill_tokens, min(args.steps, 64),
+                                         args.warmup, pk, gen, say)
+        print(json.dumps({"impl": "ours", "metric": "Sisadra beside its closest designs at equal size: decode and prefill tok/s, "
                           "per-kernel microseconds per launch", "dtype": "bf16", "data": "synthetic", "peak": tag,
                           "peaks": {"hbm_gbs": pk["hbm_gbs"], "bf16_tflops": pk["bf16_tflops"]},
                           "compare": result, "clocks": clocks.summary()}))
